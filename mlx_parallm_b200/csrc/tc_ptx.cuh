@@ -78,8 +78,8 @@ __device__ __forceinline__ void umma_f16_ts(uint32_t d_tmem, uint32_t a_tmem, ui
       : "memory");
 }
 // All eight MMAs of one k-block (64 k of 2 x 128 weight rows) in one block: the issuing warp is ONE serial instruction
-// stream for the whole CTA (measured: ~96 SASS instructions per k-block, mostly descriptor arithmetic and R2UR moves,
-// were what bounded the kernel at ~3.7 TB/s), so the per-MMA operands are formed with the fewest adds possible:
+// stream for the whole CTA (measured: forming every descriptor anew bounded the kernel at ~3.7 TB/s), so the per-MMA
+// operands are formed with the fewest adds possible:
 //   A slices at a, a+8, ..., a+56 TMEM columns (block 0: 0..24, block 1: 32..56), B descriptors at b, b+2, b+4, b+6
 //   (16-byte units: 32 bytes = 16 k per MMA).  acc = 0 clears D on the first slice of each block.
 // The two blocks' MMAs ALTERNATE: consecutive tcgen05.mma into the SAME accumulator are a dependent chain (one every
