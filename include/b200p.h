@@ -270,18 +270,20 @@ enum {
   B200P_GEMM_STORE = 0,      /* y[M,N] (dtype) = acc                                                             */
   B200P_GEMM_STORE_F32 = 1,  /* y[M,N] (float) = acc                                                             */
   B200P_GEMM_GLU_CLAMP = 2,  /* rows 2i / 2i+1 of w are gate_i / up_i: y[M,N/2] (dtype) = g * sigmoid(1.702 g) * (u + 1),
-                                g = min(gate, limit), u = clamp(up, -limit, limit)                                  */
+                                g = min(gate, act_a), u = clamp(up, -act_a, act_a)                                  */
   B200P_GEMM_GLU_GELU_TANH = 3, /* same row pairs: y = gelu_tanh(gate) * up                                          */
   B200P_GEMM_GLU_SILU = 4,   /* same row pairs: y = gate * sigmoid(gate) * up                                       */
-  B200P_GEMM_RELU_SQ = 5     /* y[M,N] (dtype) = max(acc, 0)^2: the hidden units of an ungated feed-forward           */
+  B200P_GEMM_RELU_SQ = 5,    /* y[M,N] (dtype) = max(acc, 0)^2: the hidden units of an ungated feed-forward           */
+  B200P_GEMM_XIELU = 6       /* y[M,N] (dtype) = act_a z^2 + z / 2 (z > 0), act_b (e^z - 1 - z) + z / 2 (z <= 0), z = acc */
 };
-/* y = x . w^T, x [M,K] and w [N,K] in `dtype` (row strides ldx / ldw elements), fp32 accumulation; `batch` independent
+/* act_a / act_b: the epilogue's constants (0 where it has none).
+ * y = x . w^T, x [M,K] and w [N,K] in `dtype` (row strides ldx / ldw elements), fp32 accumulation; `batch` independent
  * products at element strides stride_x / stride_w / stride_y.  B200P_F32 runs true fp32 FMAs in ascending k.  16-bit calls
  * with K % 8 == 0 and 16-byte aligned rows take the tensor-core tile kernels (more than 8 rows) or the row-streaming kernel;
  * everything else takes a generic kernel. */
 int b200p_gemm(const void* x, const void* w, void* y, int64_t M, int64_t N, int64_t K, int64_t ldx, int64_t ldw, int64_t ldy,
-               int64_t batch, int64_t stride_x, int64_t stride_w, int64_t stride_y, int dtype, int epilogue, float limit,
-               void* stream);
+               int64_t batch, int64_t stride_x, int64_t stride_w, int64_t stride_y, int dtype, int epilogue, float act_a,
+               float act_b, void* stream);
 
 /* Grouped product (the experts of a mixture): group z < groups multiplies the rows [seg[z], seg[z+1]) of x (and writes the same
  * rows of y) by its own weight block w + z * stride_w ([N, K]); seg is a DEVICE array of groups + 1 ascending offsets and
@@ -289,7 +291,7 @@ int b200p_gemm(const void* x, const void* w, void* y, int64_t M, int64_t N, int6
  * total_rows = rows of x and y (seg[groups] <= total_rows).  16-bit calls of more than 64 rows per group run on tcgen05. */
 int b200p_gemm_grouped(const void* x, const void* w, void* y, const int32_t* seg, int64_t total_rows, int64_t max_rows, int64_t N, int64_t K,
                        int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t stride_w, int dtype, int epilogue,
-                       float limit, void* stream);
+                       float act_a, float act_b, void* stream);
 
 /* 0 (default): calls of 9 rows and more run on tcgen05 (TMA-fed shared-memory operands, TMEM accumulators; up to 64 rows with the
  * weights on the MMA's M side and K split where the output is narrow, which adds fp32 partial sums in no fixed order) and fall
@@ -402,10 +404,39 @@ int b200p_moe_gather(const void* x, const int32_t* token_of, void* xs, int64_t s
 int b200p_moe_route_sigmoid(const float* logits, int64_t ldl, const float* correction, int32_t* ids, float* wts, int32_t* seg,
                             int32_t* slot_of, int32_t* token_of, int64_t M, int E, int top, int count, int keep, float scale,
                             void* stream);
-/* The same outputs from plain sigmoid scores: the `top` largest s = sigmoid(logits) are picked (ties to the smaller index) and
- * wts are those scores as they are, not renormalised. */
+/* The same outputs from plain scores: the `top` largest s = sigmoid(logits), or (softmax != 0) s = softmax(logits) over all
+ * experts, are picked (ties to the smaller index) and wts are those scores as they are, not renormalised. */
 int b200p_moe_route_scores(const float* logits, int64_t ldl, int32_t* ids, float* wts, int32_t* seg, int32_t* slot_of,
-                           int32_t* token_of, int64_t M, int E, int top, void* stream);
+                           int32_t* token_of, int64_t M, int E, int top, int softmax, void* stream);
+/* Residual step of designs whose sublayers are normed on their output only, with an optional weighted sum over the embedding
+ * output and all layers' results ("depth average").  Per token, fp32: x = h + rms_norm(y) w (y NULL: x = rms_norm(h) w);
+ * stack[t, slot] = x (slot >= 0; stack [M, slots, W]); h = sum_{j < n-1} a[j] stack[t, j] + a[n-1] x (a NULL: h = x);
+ * raw_out = h in `dtype` (NULL: not written). */
+int b200p_post_norm_step(const float* y, const float* w, float* h, float* stack, int64_t slots, int slot, const float* a, int n,
+                         void* raw_out, int64_t M, int64_t W, float eps, int dtype, void* stream);
+
+/* Attention whose heads' scores are mixed by a matrix before the softmax.  Preparation: proj columns [q | k | v] plus `bias`
+ * (indexed by the same columns; NULL: none); q and k rms-normed over their WHOLE rows with weights wq [H dk] / wk [G dk] (NULL: not
+ * normed); the first 2 n_rot dimensions of every head rotated by position * rates[i], cos and sin times `mag`, dimension i paired
+ * with i + n_rot (pairs 0) or 2i with 2i + 1 (pairs 1); q_out [M, H dk] fp32 = q * scale; k, v into the caches
+ * [rows, G, Tcap, dk] / [rows, G, Tcap, dv] at (t_row, t_pos). */
+int b200p_mix_attn_prep(const float* proj, int64_t ldp, int64_t col_q, int64_t col_k, int64_t col_v, const float* bias, const float* wq,
+                        const float* wk, float eps, const float* rates, int n_rot, float mag, int pairs, float scale, float* q_out,
+                        void* kcache, void* vcache, int64_t Tcap, const int32_t* t_row, const int32_t* t_pos, int64_t M, int H, int G,
+                        int dk, int dv, int dtype, void* stream);
+/* out[t, h] = softmax_j(sum_g talk[h, g] q_g . k_j) v_j over 0 <= position - j < window (0: every j <= position), the denominator
+ * also holding exp(sink[h]) (NULL: no sink).  talk fp32 [H, H]; 16-bit calls need talk exact in 11 significant bits (as a matrix
+ * stored in 16 bits is).  Prompts of 16-bit models (key and value sizes 64 / 128, up to 16 heads, or up to 32 whose key heads serve
+ * an even number) run on the tile kernel; the rest on the per-token kernel, whose decode steps (max_n 1) split the keys over CTAs
+ * given b200p_mix_attn_workspace_bytes of workspace. */
+int b200p_mix_attn(const float* q, const void* kcache, const void* vcache, int64_t Tcap, const int32_t* t_row, const int32_t* t_pos,
+                   const int32_t* cu, const int32_t* rows, int nb, int max_n, const float* talk, const float* sink, int64_t window,
+                   void* out, int64_t ld_out, int64_t M, int H, int G, int dk, int dv, int dtype, void* workspace,
+                   size_t workspace_bytes, void* stream);
+size_t b200p_mix_attn_workspace_bytes(int64_t nb, int H, int dv);
+/* 0, or 100 * heads per warp + keys per chunk of the tile kernel for these sizes */
+int b200p_mix_attn_tiles_supported(int H, int G, int dk, int dv, int dtype);
+
 /* xs[slot_of[t, k], :] = wts[t, k] * x[t, :] (fp32 product rounded to `dtype`): routing weights that multiply the experts' inputs */
 int b200p_moe_scatter_scaled(const void* x, const int32_t* slot_of, const float* wts, void* xs, int64_t M, int64_t W, int top,
                              int dtype, void* stream);

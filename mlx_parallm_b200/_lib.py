@@ -64,7 +64,7 @@ SIGNATURES = {
     "b200p_peer_allgather": (_i32, [_vp, _vp, _i32, _i32, _vp, _i64, _vp]),
     "b200p_peer_status": (_i32, [_vp, _vp, _vp]),
     # dense linear layers, ragged batches, gated delta rule, latent attention
-    "b200p_gemm": (_i32, [_vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i32, _i32, _f32, _vp]),
+    "b200p_gemm": (_i32, [_vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i32, _i32, _f32, _f32, _vp]),
     "b200p_gemm_set_path": (_i32, [_i32]),
     "b200p_gemm_tc_fault": (_i32, []),
     "b200p_ragged_plan": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _i32, _i64, _vp]),
@@ -78,7 +78,7 @@ SIGNATURES = {
     "b200p_delta_scan": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i32, _i32, _i32, _i32, _i32, _i32, _vp]),
     "b200p_delta_out": (_i32, [_vp, _vp, _i64, _vp, _vp, _i64, _i64, _i32, _i32, _f32, _i32, _f32, _i32, _vp]),
     "b200p_linear_attn_prep": (_i32, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _vp]),
-    "b200p_gemm_grouped": (_i32, [_vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i32, _i32, _f32, _vp]),
+    "b200p_gemm_grouped": (_i32, [_vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i32, _i32, _f32, _f32, _vp]),
     "b200p_residual_add_norm": (_i32, [_vp, _vp, _f32, _vp, _f32, _vp, _vp, _vp, _i64, _i64, _i64, _f32, _i32, _vp]),
     "b200p_cast_columns": (_i32, [_vp, _i64, _vp, _i64, _i64, _i64, _i32, _vp]),
     "b200p_sink_attn_prep": (_i32, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _f32, _f32, _f32, _f32, _vp, _vp, _vp, _i64, _vp, _vp,
@@ -91,7 +91,7 @@ SIGNATURES = {
     "b200p_moe_gather": (_i32, [_vp, _vp, _vp, _i64, _i64, _i32, _vp]),
     "b200p_moe_route_sigmoid": (_i32, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _f32, _vp]),
     "b200p_moe_combine": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _i64, _i64, _i32, _vp]),
-    "b200p_moe_route_scores": (_i32, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _vp]),
+    "b200p_moe_route_scores": (_i32, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _vp]),
     "b200p_moe_scatter_scaled": (_i32, [_vp, _vp, _vp, _vp, _i64, _i64, _i32, _i32, _vp]),
     "b200p_ssm_prep": (_i32, [_vp, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32,
                               _i32, _i32, _i32, _vp]),
@@ -120,6 +120,13 @@ SIGNATURES = {
                                 _i32, _vp]),
     "b200p_canon_conv": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i32, _i32, _vp]),
     "b200p_tanh_norm": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _i64, _i32, _vp]),
+    "b200p_post_norm_step": (_i32, [_vp, _vp, _vp, _vp, _i64, _i32, _vp, _i32, _vp, _i64, _i64, _f32, _i32, _vp]),
+    "b200p_mix_attn_prep": (_i32, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _f32, _vp, _i32, _f32, _i32, _f32, _vp, _vp, _vp, _i64, _vp,
+                                   _vp, _i64, _i32, _i32, _i32, _i32, _i32, _vp]),
+    "b200p_mix_attn": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i32, _i32, _vp, _vp, _i64, _vp, _i64, _i64, _i32, _i32, _i32, _i32,
+                              _i32, _vp, _sz, _vp]),
+    "b200p_mix_attn_workspace_bytes": (_sz, [_i64, _i32, _i32]),
+    "b200p_mix_attn_tiles_supported": (_i32, [_i32, _i32, _i32, _i32, _i32]),
 }
 
 # Translation units a model family needs (csrc/*.cu): the library can be linked from a subset, so that a fresh checkout
@@ -130,8 +137,9 @@ UNIT_SETS = {
     "sequence_ssm": ("runtime", "dense_gemm", "dense_gemm_tc", "ragged", "delta_rule", "ssm", "diff_attn", "moe", "sampler"),
     "sequence_hyper": ("runtime", "dense_gemm", "dense_gemm_tc", "ragged", "hyper", "delta_rule", "latent_attn", "sink_attn", "moe",
                        "sampler"),
+    "sequence_post": ("runtime", "dense_gemm", "dense_gemm_tc", "ragged", "post_norm", "latent_attn", "mix_attn", "moe", "sampler"),
 }
-GEMM_STORE, GEMM_STORE_F32, GEMM_GLU_CLAMP, GEMM_GLU_GELU_TANH, GEMM_GLU_SILU, GEMM_RELU_SQ = 0, 1, 2, 3, 4, 5
+GEMM_STORE, GEMM_STORE_F32, GEMM_GLU_CLAMP, GEMM_GLU_GELU_TANH, GEMM_GLU_SILU, GEMM_RELU_SQ, GEMM_XIELU = 0, 1, 2, 3, 4, 5, 6
 
 
 def gemm_is_gated(epilogue: int) -> bool:

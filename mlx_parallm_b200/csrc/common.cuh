@@ -74,15 +74,19 @@ __device__ __forceinline__ float gelu_tanh_unit(float z) {
 }
 __device__ __forceinline__ bool gemm_epi_is_glu(int epi) { return epi >= B200P_GEMM_GLU_CLAMP && epi <= B200P_GEMM_GLU_SILU; }
 // value stored by the ungated epilogues that write the storage type: the accumulator itself, or an activation of it
-__device__ __forceinline__ float gemm_store_act(float v, int epi) {
+// (act: the epilogue's constants)
+__device__ __forceinline__ float gemm_store_act(float v, int epi, float2 act) {
   if (epi == B200P_GEMM_RELU_SQ) {
     v = fmaxf(v, 0.f);
     return v * v;
   }
+  if (epi == B200P_GEMM_XIELU)       // act.x v^2 + v / 2 above zero, act.y (e^v - 1 - v) + v / 2 below: expm1f keeps small |v| exact
+    return v > 0.f ? fmaf(act.x * v, v, 0.5f * v) : fmaf(act.y, expm1f(v) - v, 0.5f * v);
   return v;
 }
-__device__ __forceinline__ float glu_unit(float gate, float up, int epi, float limit) {
+__device__ __forceinline__ float glu_unit(float gate, float up, int epi, float2 act) {
   if (epi == B200P_GEMM_GLU_CLAMP) {
+    const float limit = act.x;
     const float g = fminf(gate, limit);
     const float u = fminf(fmaxf(up, -limit), limit);
     return g / (1.f + __expf(-1.702f * g)) * (u + 1.f);

@@ -16,10 +16,10 @@ namespace b200p {
 // dense_gemm_tc.cu: B200P_OK, an error, or 1 = "not a shape for the tcgen05 kernel"
 template <typename T>
 int gemm_tc_launch(const T* x, const T* w, void* y, int64_t M, int64_t N, int64_t K, int64_t ldx, int64_t ldw, int64_t ldy,
-                   int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float limit, cudaStream_t st);
+                   int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float2 act, cudaStream_t st);
 template <typename T>
 int gemm_tc_launch_grouped(const T* x, const T* w, void* y, const int32_t* seg, int64_t total_rows, int64_t max_rows, int64_t N,
-                           int64_t K, int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t sw, int epi, float limit,
+                           int64_t K, int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t sw, int epi, float2 act,
                            cudaStream_t st);
 // 0: tcgen05 from 9 rows up (its decode variant streams the weights 1.0-2.3x faster than gemm_stream_kernel at 16 rows, 1.1-2.6x at
 //    32, 1.6-4.4x at 64), the mma.sync kernels where it declines; 1: mma.sync kernels only; 2: the same as 0
@@ -29,17 +29,17 @@ static int g_gemm_path = 0;
 // value pair (even column n, odd column n+1) of one output row
 template <typename T>
 __device__ __forceinline__ void gemm_store_pair(void* y, int64_t row_off, int64_t n, int64_t N, float v0, float v1, int epi,
-                                                float limit) {
+                                                float2 act) {
   if (epi == B200P_GEMM_STORE_F32) {
     float* p = reinterpret_cast<float*>(y) + row_off;
     if (n < N) p[n] = v0;
     if (n + 1 < N) p[n + 1] = v1;
   } else if (!gemm_epi_is_glu(epi)) {
     T* p = reinterpret_cast<T*>(y) + row_off;
-    if (n < N) p[n] = Tr<T>::from_f(gemm_store_act(v0, epi));
-    if (n + 1 < N) p[n + 1] = Tr<T>::from_f(gemm_store_act(v1, epi));
+    if (n < N) p[n] = Tr<T>::from_f(gemm_store_act(v0, epi, act));
+    if (n + 1 < N) p[n + 1] = Tr<T>::from_f(gemm_store_act(v1, epi, act));
   } else {  // gated units: v0 = gate, v1 = up of hidden unit n / 2
-    if (n + 1 < N) reinterpret_cast<T*>(y)[row_off + (n >> 1)] = Tr<T>::from_f(glu_unit(v0, v1, epi, limit));
+    if (n + 1 < N) reinterpret_cast<T*>(y)[row_off + (n >> 1)] = Tr<T>::from_f(glu_unit(v0, v1, epi, act));
   }
 }
 
@@ -64,7 +64,7 @@ constexpr int GS_BM = 64, GS_BN = 64, GS_BK = 16;
 template <typename T>
 __global__ void __launch_bounds__(256)
 gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __restrict__ y, int64_t M, int64_t N, int64_t K,
-                 int64_t ldx, int64_t ldw, int64_t ldy, int64_t sx, int64_t sw, int64_t sy, int epi, float limit,
+                 int64_t ldx, int64_t ldw, int64_t ldy, int64_t sx, int64_t sw, int64_t sy, int epi, float2 act,
                  const int32_t* __restrict__ seg) {
   __shared__ float xs[GS_BK][GS_BM + 4];
   __shared__ float ws[GS_BK][GS_BN + 4];
@@ -106,7 +106,7 @@ gemm_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __restr
     if (m >= M) continue;
     const int64_t off = ybase + m * ldy;
 #pragma unroll
-    for (int j = 0; j < 4; j += 2) gemm_store_pair<T>(y, off, n0 + tx * 4 + j, N, acc[i][j], acc[i][j + 1], epi, limit);
+    for (int j = 0; j < 4; j += 2) gemm_store_pair<T>(y, off, n0 + tx * 4 + j, N, acc[i][j], acc[i][j + 1], epi, act);
   }
 }
 
@@ -119,7 +119,7 @@ constexpr int GM_PAD = 8;
 template <typename T, int WM, int WN, int WTM, int WTN, int BK, int STAGES>
 __global__ void __launch_bounds__(WM * WN * 32)
 gemm_mma_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __restrict__ y, int64_t M, int64_t N, int64_t K,
-                int64_t ldx, int64_t ldw, int64_t ldy, int64_t sx, int64_t sw, int64_t sy, int epi, float limit,
+                int64_t ldx, int64_t ldw, int64_t ldy, int64_t sx, int64_t sw, int64_t sy, int epi, float2 act,
                 const int32_t* __restrict__ seg) {
   constexpr int BM = WM * WTM, BN = WN * WTN, NT = WM * WN * 32, LDS = BK + GM_PAD, MI = WTM / 16, NJ = WTN / 8;
   static_assert(WTM % 16 == 0 && WTN % 16 == 0 && BK % 16 == 0, "warp blocks are made of 16 x 16 pieces");
@@ -197,13 +197,13 @@ gemm_mma_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __restri
       const int64_t off = ybase + m * ldy;
 #pragma unroll
       for (int j = 0; j < NJ; ++j)
-        gemm_store_pair<T>(y, off, n0 + wn * WTN + j * 8 + (lane & 3) * 2, N, acc[i][j][hf * 2], acc[i][j][hf * 2 + 1], epi, limit);
+        gemm_store_pair<T>(y, off, n0 + wn * WTN + j * 8 + (lane & 3) * 2, N, acc[i][j][hf * 2], acc[i][j][hf * 2 + 1], epi, act);
     }
 }
 
 template <typename T, int WM, int WN, int WTM, int WTN, int BK, int STAGES>
 static int gemm_mma_launch(const T* x, const T* w, void* y, int64_t M, int64_t N, int64_t K, int64_t ldx, int64_t ldw, int64_t ldy,
-                           int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float limit, cudaStream_t st,
+                           int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float2 act, cudaStream_t st,
                            const int32_t* seg = nullptr) {
   constexpr int BM = WM * WTM, BN = WN * WTN;
   constexpr size_t smem = (size_t)STAGES * (BM + BN) * (BK + GM_PAD) * sizeof(T);
@@ -217,7 +217,7 @@ static int gemm_mma_launch(const T* x, const T* w, void* y, int64_t M, int64_t N
     }
   }
   dim3 grid((unsigned)((N + BN - 1) / BN), (unsigned)((M + BM - 1) / BM), (unsigned)batch);
-  kern<<<grid, WM * WN * 32, smem, st>>>(x, w, y, M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, limit, seg);
+  kern<<<grid, WM * WN * 32, smem, st>>>(x, w, y, M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, act, seg);
   B200P_LAUNCH_CHECK("gemm_mma_kernel");
   return B200P_OK;
 }
@@ -228,7 +228,7 @@ constexpr int GEMV_MAX_M = 8;
 template <typename T, int MR>
 __global__ void __launch_bounds__(256)
 gemv_rows_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __restrict__ y, int M, int64_t N, int64_t K, int64_t ldx,
-                 int64_t ldw, int64_t ldy, int64_t sx, int64_t sw, int64_t sy, int epi, float limit) {
+                 int64_t ldw, int64_t ldy, int64_t sx, int64_t sw, int64_t sy, int epi, float2 act) {
   const int64_t z = blockIdx.z;
   x += z * sx;
   w += z * sw;
@@ -273,7 +273,7 @@ gemv_rows_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __restr
   if (lane == 0) {
 #pragma unroll
     for (int m = 0; m < MR; ++m)
-      if (m < M) gemm_store_pair<T>(y, z * sy + (int64_t)m * ldy, n, N, a0[m], a1[m], epi, limit);
+      if (m < M) gemm_store_pair<T>(y, z * sy + (int64_t)m * ldy, n, N, a0[m], a1[m], epi, act);
   }
 }
 
@@ -288,7 +288,7 @@ constexpr int GK_SLICES = 4, GK_THREADS = 256;
 template <typename T, int MT>     // MT m16 tiles: rows <= 16 * MT
 __global__ void __launch_bounds__(GK_THREADS)
 gemm_stream_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __restrict__ y, int M, int64_t N, int64_t K, int64_t ldx,
-                   int64_t ldw, int64_t ldy, int64_t sx, int64_t sw, int64_t sy, int epi, float limit,
+                   int64_t ldw, int64_t ldy, int64_t sx, int64_t sw, int64_t sy, int epi, float2 act,
                    const int32_t* __restrict__ seg) {
   __shared__ float red[GK_SLICES][2][MT][32][4];
   const int64_t z = blockIdx.z;
@@ -345,53 +345,53 @@ gemm_stream_kernel(const T* __restrict__ x, const T* __restrict__ w, void* __res
       const int m = i * 16 + (lane >> 2) + hf * 8;
       if (m < M)
         gemm_store_pair<T>(y, ybase + (int64_t)m * ldy, (int64_t)blockIdx.x * 16 + nt * 8 + (lane & 3) * 2, N, v[hf * 2], v[hf * 2 + 1],
-                           epi, limit);
+                           epi, act);
     }
   }
 }
 
 template <typename T>
 static int gemm_dispatch(const void* x, const void* w, void* y, int64_t M, int64_t N, int64_t K, int64_t ldx, int64_t ldw,
-                         int64_t ldy, int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float limit, bool fast_ok,
+                         int64_t ldy, int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float2 act, bool fast_ok,
                          cudaStream_t st) {
   const T* xp = (const T*)x;
   const T* wp = (const T*)w;
   if (fast_ok && M <= GEMV_MAX_M) {
     dim3 grid((unsigned)((N + 15) / 16), 1, (unsigned)batch);
-    if (M <= 2) gemv_rows_kernel<T, 2><<<grid, 256, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, limit);
-    else if (M <= 4) gemv_rows_kernel<T, 4><<<grid, 256, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, limit);
-    else gemv_rows_kernel<T, 8><<<grid, 256, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, limit);
+    if (M <= 2) gemv_rows_kernel<T, 2><<<grid, 256, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, act);
+    else if (M <= 4) gemv_rows_kernel<T, 4><<<grid, 256, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, act);
+    else gemv_rows_kernel<T, 8><<<grid, 256, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, act);
     B200P_LAUNCH_CHECK("gemv_rows_kernel");
     return B200P_OK;
   }
   if (fast_ok) {
     if constexpr (!std::is_same<T, float>::value) {
       if (M <= 64 && g_gemm_path != 1) {
-        const int rc = gemm_tc_launch<T>(xp, wp, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, limit, st);
+        const int rc = gemm_tc_launch<T>(xp, wp, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, act, st);
         if (rc != 1) return rc;
       }
     }
     if (M <= 64) {
       dim3 grid((unsigned)((N + 15) / 16), 1, (unsigned)batch);
-      if (M <= 16) gemm_stream_kernel<T, 1><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, limit, nullptr);
-      else if (M <= 32) gemm_stream_kernel<T, 2><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, limit, nullptr);
-      else gemm_stream_kernel<T, 4><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, limit, nullptr);
+      if (M <= 16) gemm_stream_kernel<T, 1><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, act, nullptr);
+      else if (M <= 32) gemm_stream_kernel<T, 2><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, act, nullptr);
+      else gemm_stream_kernel<T, 4><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, (int)M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, act, nullptr);
       B200P_LAUNCH_CHECK("gemm_stream_kernel");
       return B200P_OK;
     }
     if constexpr (!std::is_same<T, float>::value) {
       if (g_gemm_path != 1) {
-        const int rc = gemm_tc_launch<T>(xp, wp, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, limit, st);
+        const int rc = gemm_tc_launch<T>(xp, wp, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, act, st);
         if (rc != 1) return rc;
       }
     }
     // mma.sync: 128 x 128 tiles once that grid covers most of the GPU's SMs, 64 x 64 below
     const int64_t big = ((M + 127) / 128) * ((N + 127) / 128) * batch;
-    if (big >= 96) return gemm_mma_launch<T, 2, 2, 64, 64, 32, 4>(xp, wp, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, limit, st);
-    return gemm_mma_launch<T, 2, 2, 32, 32, 32, 3>(xp, wp, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, limit, st);
+    if (big >= 96) return gemm_mma_launch<T, 2, 2, 64, 64, 32, 4>(xp, wp, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, act, st);
+    return gemm_mma_launch<T, 2, 2, 32, 32, 32, 3>(xp, wp, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, act, st);
   }
   dim3 grid((unsigned)((N + GS_BN - 1) / GS_BN), (unsigned)((M + GS_BM - 1) / GS_BM), (unsigned)batch);
-  gemm_simt_kernel<T><<<grid, 256, 0, st>>>(xp, wp, y, M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, limit, nullptr);
+  gemm_simt_kernel<T><<<grid, 256, 0, st>>>(xp, wp, y, M, N, K, ldx, ldw, ldy, sx, sw, sy, epi, act, nullptr);
   B200P_LAUNCH_CHECK("gemm_simt_kernel");
   return B200P_OK;
 }
@@ -399,29 +399,29 @@ static int gemm_dispatch(const void* x, const void* w, void* y, int64_t M, int64
 // groups of at most max_rows rows each: the row-streaming kernel while a group fits its 64 rows, 64 x 64 tiles beyond
 template <typename T>
 static int gemm_grouped_dispatch(const void* x, const void* w, void* y, const int32_t* seg, int64_t total_rows, int64_t max_rows, int64_t N, int64_t K,
-                                 int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t sw, int epi, float limit, bool fast_ok,
+                                 int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t sw, int epi, float2 act, bool fast_ok,
                                  cudaStream_t st) {
   const T* xp = (const T*)x;
   const T* wp = (const T*)w;
   if (fast_ok && max_rows <= 64) {
     dim3 grid((unsigned)((N + 15) / 16), 1, (unsigned)groups);
-    if (max_rows <= 16) gemm_stream_kernel<T, 1><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, 0, N, K, ldx, ldw, ldy, 0, sw, 0, epi, limit, seg);
-    else if (max_rows <= 32) gemm_stream_kernel<T, 2><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, 0, N, K, ldx, ldw, ldy, 0, sw, 0, epi, limit, seg);
-    else gemm_stream_kernel<T, 4><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, 0, N, K, ldx, ldw, ldy, 0, sw, 0, epi, limit, seg);
+    if (max_rows <= 16) gemm_stream_kernel<T, 1><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, 0, N, K, ldx, ldw, ldy, 0, sw, 0, epi, act, seg);
+    else if (max_rows <= 32) gemm_stream_kernel<T, 2><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, 0, N, K, ldx, ldw, ldy, 0, sw, 0, epi, act, seg);
+    else gemm_stream_kernel<T, 4><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, 0, N, K, ldx, ldw, ldy, 0, sw, 0, epi, act, seg);
     B200P_LAUNCH_CHECK("gemm_stream_kernel");
     return B200P_OK;
   }
   if (fast_ok) {
     if constexpr (!std::is_same<T, float>::value) {
       if (g_gemm_path != 1) {
-        const int rc = gemm_tc_launch_grouped<T>(xp, wp, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, sw, epi, limit, st);
+        const int rc = gemm_tc_launch_grouped<T>(xp, wp, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, sw, epi, act, st);
         if (rc != 1) return rc;
       }
     }
-    return gemm_mma_launch<T, 2, 2, 32, 32, 32, 3>(xp, wp, y, max_rows, N, K, ldx, ldw, ldy, groups, 0, sw, 0, epi, limit, st, seg);
+    return gemm_mma_launch<T, 2, 2, 32, 32, 32, 3>(xp, wp, y, max_rows, N, K, ldx, ldw, ldy, groups, 0, sw, 0, epi, act, st, seg);
   }
   dim3 grid((unsigned)((N + GS_BN - 1) / GS_BN), (unsigned)((max_rows + GS_BM - 1) / GS_BM), (unsigned)groups);
-  gemm_simt_kernel<T><<<grid, 256, 0, st>>>(xp, wp, y, max_rows, N, K, ldx, ldw, ldy, 0, sw, 0, epi, limit, seg);
+  gemm_simt_kernel<T><<<grid, 256, 0, st>>>(xp, wp, y, max_rows, N, K, ldx, ldw, ldy, 0, sw, 0, epi, act, seg);
   B200P_LAUNCH_CHECK("gemm_simt_kernel");
   return B200P_OK;
 }
@@ -430,12 +430,12 @@ static int gemm_grouped_dispatch(const void* x, const void* w, void* y, const in
 
 extern "C" int b200p_gemm_grouped(const void* x, const void* w, void* y, const int32_t* seg, int64_t total_rows, int64_t max_rows, int64_t N, int64_t K,
                                   int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t stride_w, int dtype, int epilogue,
-                                  float limit, void* stream) {
+                                  float act_a, float act_b, void* stream) {
   using namespace b200p;
   B200P_REQUIRE(x && w && y && seg, B200P_ERR_ARG, "null pointer");
   B200P_REQUIRE(total_rows >= max_rows, B200P_ERR_ARG, "x has fewer rows than a group may have");
   B200P_REQUIRE(max_rows >= 0 && N > 0 && K > 0 && groups > 0 && groups < 65536 && ldx >= K && ldw >= K, B200P_ERR_ARG, "bad GEMM shape");
-  B200P_REQUIRE(epilogue >= B200P_GEMM_STORE && epilogue <= B200P_GEMM_RELU_SQ, B200P_ERR_ARG, "unknown epilogue %d", epilogue);
+  B200P_REQUIRE(epilogue >= B200P_GEMM_STORE && epilogue <= B200P_GEMM_XIELU, B200P_ERR_ARG, "unknown epilogue %d", epilogue);
   B200P_REQUIRE(epilogue < B200P_GEMM_GLU_CLAMP || epilogue > B200P_GEMM_GLU_SILU || N % 2 == 0, B200P_ERR_ARG, "the gated epilogue needs gate / up row pairs");
   B200P_REQUIRE((max_rows + 63) / 64 < 65536, B200P_ERR_ARG, "grid too large");
   if (max_rows == 0) return B200P_OK;
@@ -444,11 +444,11 @@ extern "C" int b200p_gemm_grouped(const void* x, const void* w, void* y, const i
                        aligned(w, 16);
   switch (dtype) {
     case B200P_F32:
-      return gemm_grouped_dispatch<float>(x, w, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, stride_w, epilogue, limit, false, st);
+      return gemm_grouped_dispatch<float>(x, w, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, stride_w, epilogue, {act_a, act_b}, false, st);
     case B200P_F16:
-      return gemm_grouped_dispatch<__half>(x, w, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, stride_w, epilogue, limit, fast_ok, st);
+      return gemm_grouped_dispatch<__half>(x, w, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, stride_w, epilogue, {act_a, act_b}, fast_ok, st);
     case B200P_BF16:
-      return gemm_grouped_dispatch<__nv_bfloat16>(x, w, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, stride_w, epilogue, limit,
+      return gemm_grouped_dispatch<__nv_bfloat16>(x, w, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, stride_w, epilogue, {act_a, act_b},
                                                   fast_ok, st);
     default:
       set_error("bad dtype %d", dtype);
@@ -463,11 +463,11 @@ extern "C" int b200p_gemm_set_path(int path) {
 
 extern "C" int b200p_gemm(const void* x, const void* w, void* y, int64_t M, int64_t N, int64_t K, int64_t ldx, int64_t ldw,
                           int64_t ldy, int64_t batch, int64_t stride_x, int64_t stride_w, int64_t stride_y, int dtype,
-                          int epilogue, float limit, void* stream) {
+                          int epilogue, float act_a, float act_b, void* stream) {
   using namespace b200p;
   B200P_REQUIRE(x && w && y, B200P_ERR_ARG, "null pointer");
   B200P_REQUIRE(M >= 0 && N > 0 && K > 0 && batch > 0 && ldx >= K && ldw >= K, B200P_ERR_ARG, "bad GEMM shape");
-  B200P_REQUIRE(epilogue >= B200P_GEMM_STORE && epilogue <= B200P_GEMM_RELU_SQ, B200P_ERR_ARG, "unknown epilogue %d", epilogue);
+  B200P_REQUIRE(epilogue >= B200P_GEMM_STORE && epilogue <= B200P_GEMM_XIELU, B200P_ERR_ARG, "unknown epilogue %d", epilogue);
   B200P_REQUIRE(epilogue < B200P_GEMM_GLU_CLAMP || epilogue > B200P_GEMM_GLU_SILU || N % 2 == 0, B200P_ERR_ARG, "the gated epilogue needs gate / up row pairs");
   B200P_REQUIRE((M + 63) / 64 < 65536 && batch < 65536, B200P_ERR_ARG, "grid too large");
   if (M == 0) return B200P_OK;
@@ -477,11 +477,11 @@ extern "C" int b200p_gemm(const void* x, const void* w, void* y, int64_t M, int6
                        stride_w % 8 == 0 && aligned(x, 16) && aligned(w, 16);
   switch (dtype) {
     case B200P_F32:
-      return gemm_dispatch<float>(x, w, y, M, N, K, ldx, ldw, ldy, batch, stride_x, stride_w, stride_y, epilogue, limit, false, st);
+      return gemm_dispatch<float>(x, w, y, M, N, K, ldx, ldw, ldy, batch, stride_x, stride_w, stride_y, epilogue, {act_a, act_b}, false, st);
     case B200P_F16:
-      return gemm_dispatch<__half>(x, w, y, M, N, K, ldx, ldw, ldy, batch, stride_x, stride_w, stride_y, epilogue, limit, fast_ok, st);
+      return gemm_dispatch<__half>(x, w, y, M, N, K, ldx, ldw, ldy, batch, stride_x, stride_w, stride_y, epilogue, {act_a, act_b}, fast_ok, st);
     case B200P_BF16:
-      return gemm_dispatch<__nv_bfloat16>(x, w, y, M, N, K, ldx, ldw, ldy, batch, stride_x, stride_w, stride_y, epilogue, limit,
+      return gemm_dispatch<__nv_bfloat16>(x, w, y, M, N, K, ldx, ldw, ldy, batch, stride_x, stride_w, stride_y, epilogue, {act_a, act_b},
                                           fast_ok, st);
     default:
       set_error("bad dtype %d", dtype);

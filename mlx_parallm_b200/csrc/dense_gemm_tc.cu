@@ -46,7 +46,7 @@ struct GemmTcParams {
   int splits, kb_per_split;      // K split over `splits` CTAs per output tile (transposed fp32 store only)
   int trans;                     // operands swapped: accumulator row = output column, accumulator column = token
   int epi, vec_ok;
-  float limit;
+  float2 act;
   // grouped products (not with trans): batch index z owns the rows [seg[z], seg[z+1]) of x and y; tiles past a group's rows are
   // skipped by every role alike; seg (device, groups + 1 offsets) is copied to shared memory first
   const int32_t* seg;
@@ -99,7 +99,7 @@ __device__ __forceinline__ void gemm_tc_store32(const GemmTcParams& p, int64_t r
   } else if (!gemm_epi_is_glu(p.epi)) {
     float a[32];
 #pragma unroll
-    for (int i = 0; i < 32; ++i) a[i] = gemm_store_act(v[i], p.epi);
+    for (int i = 0; i < 32; ++i) a[i] = gemm_store_act(v[i], p.epi, p.act);
     T* dst = reinterpret_cast<T*>(p.y) + row_off + n0;
     if (p.vec_ok && n0 + 32 <= p.N) {
 #pragma unroll
@@ -119,7 +119,7 @@ __device__ __forceinline__ void gemm_tc_store32(const GemmTcParams& p, int64_t r
   } else {  // gated units: columns 2i / 2i+1 are gate_i / up_i
     float a[16];
 #pragma unroll
-    for (int i = 0; i < 16; ++i) a[i] = glu_unit(v[2 * i], v[2 * i + 1], p.epi, p.limit);
+    for (int i = 0; i < 16; ++i) a[i] = glu_unit(v[2 * i], v[2 * i + 1], p.epi, p.act);
     T* dst = reinterpret_cast<T*>(p.y) + row_off + (n0 >> 1);
     if (p.vec_ok && n0 + 32 <= p.N) {
 #pragma unroll
@@ -148,7 +148,7 @@ __device__ __forceinline__ void gemm_tc_store32_trans(const GemmTcParams& p, int
     for (int i = 0; i < 32; ++i) {
       const float other = __shfl_xor_sync(0xffffffffu, v[i], 1);
       if (!(threadIdx.x & 1) && n + 1 < p.M && tok0 + i < p.N)
-        reinterpret_cast<T*>(p.y)[z_off + (tok0 + i) * p.ldy + (n >> 1)] = Tr<T>::from_f(glu_unit(v[i], other, p.epi, p.limit));
+        reinterpret_cast<T*>(p.y)[z_off + (tok0 + i) * p.ldy + (n >> 1)] = Tr<T>::from_f(glu_unit(v[i], other, p.epi, p.act));
     }
     return;
   }
@@ -168,7 +168,7 @@ __device__ __forceinline__ void gemm_tc_store32_trans(const GemmTcParams& p, int
     T* dst = reinterpret_cast<T*>(p.y) + z_off + n;
 #pragma unroll
     for (int i = 0; i < 32; ++i)
-      if (tok0 + i < p.N) dst[(tok0 + i) * p.ldy] = Tr<T>::from_f(gemm_store_act(v[i], p.epi));
+      if (tok0 + i < p.N) dst[(tok0 + i) * p.ldy] = Tr<T>::from_f(gemm_store_act(v[i], p.epi, p.act));
   }
 }
 
@@ -388,7 +388,7 @@ static int gemm_tc_run(const CUtensorMap& tmx, const CUtensorMap& tmw, GemmTcPar
 // Up to 64 tokens: weights on the M side, tokens on the N side, transposed store, K split where the output is narrow.
 template <typename T>
 static int gemm_tc_launch_decode(TcEncodeFn enc, const T* x, const T* w, void* y, int64_t M, int64_t N, int64_t K, int64_t ldx, int64_t ldw,
-                                 int64_t ldy, int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float limit, cudaStream_t st) {
+                                 int64_t ldy, int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float2 act, cudaStream_t st) {
   const CUtensorMapDataType dt = std::is_same<T, __nv_bfloat16>::value ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
   const int bn = M <= 32 ? 32 : 64;
   CUtensorMap tma, tmb;                            // A = weights (128-row boxes), B = tokens (bn-row boxes)
@@ -415,7 +415,7 @@ static int gemm_tc_launch_decode(TcEncodeFn enc, const T* x, const T* w, void* y
   p.seg = nullptr;
   p.groups = 0;
   p.epi = epi;
-  p.limit = limit;
+  p.act = act;
   p.vec_ok = 0;
   if (p.splits > 1) {
     cudaError_t e = cudaMemsetAsync(y, 0, (size_t)M * N * sizeof(float), st);
@@ -428,11 +428,11 @@ static int gemm_tc_launch_decode(TcEncodeFn enc, const T* x, const T* w, void* y
 // Returns B200P_OK, an error, or 1 when the shape is not one this kernel takes (the caller then runs the mma.sync kernel).
 template <typename T>
 int gemm_tc_launch(const T* x, const T* w, void* y, int64_t M, int64_t N, int64_t K, int64_t ldx, int64_t ldw, int64_t ldy,
-                   int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float limit, cudaStream_t st) {
+                   int64_t batch, int64_t sx, int64_t sw, int64_t sy, int epi, float2 act, cudaStream_t st) {
   if (K < GT_BK || M >= (1ll << 31) || N >= (1ll << 31) || K >= (1ll << 31)) return 1;
   TcEncodeFn enc = gemm_tc_encode_fn();
   if (!enc) return 1;
-  if (M <= 64) return gemm_tc_launch_decode<T>(enc, x, w, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, limit, st);
+  if (M <= 64) return gemm_tc_launch_decode<T>(enc, x, w, y, M, N, K, ldx, ldw, ldy, batch, sx, sw, sy, epi, act, st);
   const int tiles_m = (int)((M + GT_BM - 1) / GT_BM);
   // widest weight tile that still gives every SM about two tiles
   const int64_t want = 2ll * sm_count();
@@ -458,7 +458,7 @@ int gemm_tc_launch(const T* x, const T* w, void* y, int64_t M, int64_t N, int64_
   p.seg = nullptr;
   p.groups = 0;
   p.epi = epi;
-  p.limit = limit;
+  p.act = act;
   const int64_t eb = epi == B200P_GEMM_STORE_F32 ? 4 : 2;
   p.vec_ok = aligned(y, 16) && (ldy * eb) % 16 == 0 && (sy * eb) % 16 == 0;
   if (bn == 256) return gemm_tc_run<T, 256, 4>(tmx, tmw, p, st);
@@ -472,7 +472,7 @@ int gemm_tc_launch(const T* x, const T* w, void* y, int64_t M, int64_t N, int64_
 // rows are not stored.
 template <typename T>
 int gemm_tc_launch_grouped(const T* x, const T* w, void* y, const int32_t* seg, int64_t total_rows, int64_t max_rows, int64_t N,
-                           int64_t K, int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t sw, int epi, float limit,
+                           int64_t K, int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t sw, int epi, float2 act,
                            cudaStream_t st) {
   if (K < GT_BK || total_rows >= (1ll << 31) || N >= (1ll << 31) || K >= (1ll << 31) || groups > GT_MAX_GROUPS) return 1;
   TcEncodeFn enc = gemm_tc_encode_fn();
@@ -497,7 +497,7 @@ int gemm_tc_launch_grouped(const T* x, const T* w, void* y, const int32_t* seg, 
   p.seg = seg;
   p.groups = (int)groups;
   p.epi = epi;
-  p.limit = limit;
+  p.act = act;
   const int64_t eb = epi == B200P_GEMM_STORE_F32 ? 4 : 2;
   p.vec_ok = aligned(y, 16) && (ldy * eb) % 16 == 0;
   if (bn == 256) return gemm_tc_run<T, 256, 4>(tmx, tmw, p, st);
@@ -505,14 +505,14 @@ int gemm_tc_launch_grouped(const T* x, const T* w, void* y, const int32_t* seg, 
   return gemm_tc_run<T, 64, 8>(tmx, tmw, p, st);
 }
 template int gemm_tc_launch_grouped<__half>(const __half*, const __half*, void*, const int32_t*, int64_t, int64_t, int64_t, int64_t, int64_t,
-                                            int64_t, int64_t, int64_t, int64_t, int, float, cudaStream_t);
+                                            int64_t, int64_t, int64_t, int64_t, int, float2, cudaStream_t);
 template int gemm_tc_launch_grouped<__nv_bfloat16>(const __nv_bfloat16*, const __nv_bfloat16*, void*, const int32_t*, int64_t, int64_t,
-                                                   int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, int, float, cudaStream_t);
+                                                   int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, int, float2, cudaStream_t);
 
 template int gemm_tc_launch<__half>(const __half*, const __half*, void*, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t,
-                                    int64_t, int64_t, int64_t, int64_t, int, float, cudaStream_t);
+                                    int64_t, int64_t, int64_t, int64_t, int, float2, cudaStream_t);
 template int gemm_tc_launch<__nv_bfloat16>(const __nv_bfloat16*, const __nv_bfloat16*, void*, int64_t, int64_t, int64_t, int64_t,
-                                           int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, int, float, cudaStream_t);
+                                           int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, int, float2, cudaStream_t);
 
 }  // namespace b200p
 

@@ -1,0 +1,662 @@
+// Attention whose heads' scores are mixed before the softmax: score_h = sum_g talk[h, g] (q_g . k_{kv(g)}), a matrix over the query
+// heads of one layer, over a ragged batch with a sliding window and a learned sink per head (one extra term exp(sink_h) in the
+// denominator).  Every head's probabilities need every head's raw scores, so one CTA holds all heads of its queries.
+//   mix_attn_prep_kernel   biases on q, k, v; q and k rms-normed as whole rows; half-split or pairwise rotation of the first
+//                          dimensions of every head; q scaled, k and v into the cache at (row, position)                (per token)
+//   mix_attn_kernel        one token, all heads, fp32 throughout, any sizes; the keys optionally split over CTAs whose partial
+//                          sums attn_merge_kernel combines (decode steps)                                                (per token)
+//   mix_attn_tile_kernel   prompts of 16-bit models on mma.sync: 16 query rows per warp, one warp per head (or 8 queries of two
+//                          neighbouring heads that share a key/value head); the raw scores meet in shared memory in fp32 and are
+//                          mixed by a second matrix product (tf32 with the scores split in two, so that nothing is lost)
+// Everything from the biased projections to the softmax statistics is fp32; caches and matrix operands are in the storage type.
+#include "attn_merge.cuh"
+#include "common.cuh"
+#include "mma_util.cuh"
+
+namespace b200p {
+
+// V neighbouring channels per access (4: every head starts on a 16-byte boundary and a rotated group of 4 stays inside its half)
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+mix_attn_prep_kernel(const float* __restrict__ proj, int64_t ldp, int64_t col_q, int64_t col_k, int64_t col_v,
+                     const float* __restrict__ bias, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
+                     const float* __restrict__ rates, int n_rot, float mag, int pairs, float scale, float* __restrict__ q_out,
+                     T* __restrict__ kcache, T* __restrict__ vcache, int64_t Tcap, const int32_t* __restrict__ t_row,
+                     const int32_t* __restrict__ t_pos, int H, int G, int dk, int dv) {
+  extern __shared__ float mp_sm[];                                 // cos, sin of this position: [n_rot] each
+  __shared__ float red[2][8];
+  float* cs = mp_sm;
+  float* sn = mp_sm + n_rot;
+  const int64_t t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int64_t pos = t_pos[t], row = t_row[t];
+  const float* pt = proj + t * ldp;
+  for (int i = threadIdx.x; i < n_rot; i += blockDim.x) {
+    float s, c;
+    sincosf((float)pos * rates[i], &s, &c);
+    cs[i] = c * mag;
+    sn[i] = s * mag;
+  }
+  auto load = [&](int64_t col, float (&r)[V]) {                    // biased projection columns
+    if constexpr (V == 4) {
+      const float4 q = *reinterpret_cast<const float4*>(pt + col);
+      r[0] = q.x; r[1] = q.y; r[2] = q.z; r[3] = q.w;
+      if (bias) {
+        const float4 b = *reinterpret_cast<const float4*>(bias + col);
+        r[0] += b.x; r[1] += b.y; r[2] += b.z; r[3] += b.w;
+      }
+    } else {
+      r[0] = pt[col] + (bias ? bias[col] : 0.f);
+    }
+  };
+  const int nq = H * dk, nk = G * dk;
+  float sq = 0.f, sk = 0.f;
+  if (wq)
+    for (int c = threadIdx.x * V; c < nq; c += blockDim.x * V) {
+      float r[V];
+      load(col_q + c, r);
+#pragma unroll
+      for (int k = 0; k < V; ++k) sq = fmaf(r[k], r[k], sq);
+    }
+  if (wk)
+    for (int c = threadIdx.x * V; c < nk; c += blockDim.x * V) {
+      float r[V];
+      load(col_k + c, r);
+#pragma unroll
+      for (int k = 0; k < V; ++k) sk = fmaf(r[k], r[k], sk);
+    }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if (lane == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+  for (int i = 0; i < nw; ++i) { sq += red[0][i]; sk += red[1][i]; }
+  const float inv_q = wq ? 1.f / sqrtf(sq / (float)nq + eps) : 1.f, inv_k = wk ? 1.f / sqrtf(sk / (float)nk + eps) : 1.f;
+  const bool in_cache = pos < Tcap;                                // the host sizes the cache first; never write outside it
+  for (int c = threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
+    const bool is_q = c < nq;
+    const int cc = is_q ? c : c - nq;
+    const int head = cc / dk, i = cc % dk;
+    const int64_t col = is_q ? col_q : col_k;
+    const float* w = is_q ? wq : wk;
+    const float inv = is_q ? inv_q : inv_k;
+    float x[V];
+    load(col + cc, x);
+#pragma unroll
+    for (int k = 0; k < V; ++k) x[k] *= inv * (w ? w[cc + k] : 1.f);
+    if (i < 2 * n_rot) {                                           // rotated: u' = u cos - v sin, v' = v cos + u sin
+      const bool first = pairs ? (i & 1) == 0 : i < n_rot;
+      const int f = pairs ? i >> 1 : (first ? i : i - n_rot);
+      const int other = pairs ? cc ^ 1 : (first ? cc + n_rot : cc - n_rot);     // heads start at even columns: cc ^ 1 is the partner
+      float o[V];
+      load(col + other, o);
+#pragma unroll
+      for (int k = 0; k < V; ++k) {
+        o[k] *= inv * (w ? w[other + k] : 1.f);
+        x[k] = first ? x[k] * cs[f + k] - o[k] * sn[f + k] : x[k] * cs[f + k] + o[k] * sn[f + k];
+      }
+    }
+    if (is_q) {
+      float* d = q_out + t * nq + cc;
+      if constexpr (V == 4) *reinterpret_cast<float4*>(d) = make_float4(x[0] * scale, x[1] * scale, x[2] * scale, x[3] * scale);
+      else d[0] = x[0] * scale;
+    } else if (in_cache) {
+      T* d = kcache + ((row * G + head) * Tcap + pos) * dk + i;
+#pragma unroll
+      for (int k = 0; k < V; ++k) d[k] = Tr<T>::from_f(x[k]);
+    }
+  }
+  if (in_cache)
+    for (int c = threadIdx.x; c < G * dv; c += blockDim.x) {
+      const int g = c / dv, i = c % dv;
+      vcache[((row * G + g) * Tcap + pos) * dv + i] = Tr<T>::from_f(pt[col_v + c] + (bias ? bias[col_v + c] : 0.f));
+    }
+}
+
+// ---- one token per CTA -----------------------------------------------------------------------------------------------------
+constexpr int MX_KEYS = 32;          // keys per chunk: one per lane while scores are formed
+constexpr int MX_THREADS = 256;
+constexpr int MX_HEADS = 4;          // query heads of one key/value head scored together (they share the key's load)
+constexpr int MX_MAX_SPLITS = 16;
+constexpr int MX_SMEM_MAX = 227 * 1024;
+
+// CTA = (share of the keys blockIdx.x of gridDim.x, token blockIdx.y).  VEC elements per 16-byte piece of a cache row (1: rows that
+// are not whole pieces).  kv_block key heads are staged at a time.  part_o NULL: the whole softmax, sink included, into `out`.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(MX_THREADS)
+mix_attn_kernel(const float* __restrict__ q, const T* __restrict__ kcache, const T* __restrict__ vcache, int64_t Tcap,
+                const int32_t* __restrict__ t_row, const int32_t* __restrict__ t_pos, const float* __restrict__ talk,
+                const float* __restrict__ sink, int64_t window, T* __restrict__ out, int64_t ld_out, int H, int G, int dk, int dv,
+                float* __restrict__ part_o, float* __restrict__ part_ms, int kv_block) {
+  extern __shared__ __align__(16) uint8_t mx_smem[];
+  const int per = H / G, KP = VEC > 1 ? dk + VEC : dk + 1;          // padded key row
+  T* kst = reinterpret_cast<T*>(mx_smem);                            // [kv_block][MX_KEYS][KP]
+  float* qs = reinterpret_cast<float*>(mx_smem + ((size_t)kv_block * MX_KEYS * KP * sizeof(T) + 15) / 16 * 16);   // [H][dk]
+  float* acc = qs + H * dk;                                          // [H][dv]
+  float* tk = acc + H * dv;                                          // [H][H]
+  float* raw = tk + H * H;                                           // [H][MX_KEYS]
+  float* pr = raw + H * MX_KEYS;                                     // [H][MX_KEYS]
+  float* m_s = pr + H * MX_KEYS;                                     // [H] each: running max, sum, this chunk's rescale factor
+  float* l_s = m_s + H;
+  float* c_s = l_s + H;
+  const int64_t t = blockIdx.y;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = MX_THREADS / 32;
+  const int64_t pos = t_pos[t];
+  const T* kb = kcache + (int64_t)t_row[t] * G * Tcap * dk;
+  const T* vb = vcache + (int64_t)t_row[t] * G * Tcap * dv;
+  const bool whole = part_o == nullptr;
+  for (int i = threadIdx.x; i < H * dk; i += MX_THREADS) qs[i] = q[t * H * dk + i];
+  for (int i = threadIdx.x; i < H * dv; i += MX_THREADS) acc[i] = 0.f;
+  for (int i = threadIdx.x; i < H * H; i += MX_THREADS) tk[i] = talk[i];
+  for (int h = threadIdx.x; h < H; h += MX_THREADS) {
+    m_s[h] = whole && sink ? sink[h] : -INFINITY;
+    l_s[h] = whole && sink ? 1.f : 0.f;
+  }
+  const int64_t lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  const int64_t chunks = (pos - lo) / MX_KEYS + 1, share = (chunks + gridDim.x - 1) / gridDim.x;
+  const int64_t c_lo = blockIdx.x * share, c_hi = min(chunks, c_lo + share);
+  for (int64_t ci = c_lo; ci < c_hi; ++ci) {
+    const int64_t j0 = lo + ci * MX_KEYS;
+    const int nk = (int)min((int64_t)MX_KEYS, pos + 1 - j0);
+    for (int g0 = 0; g0 < G; g0 += kv_block) {
+      const int ng = min(kv_block, G - g0);
+      __syncthreads();                                               // the staged keys and the raw scores of the last round are used up
+      if constexpr (VEC > 1) {
+        const int pieces = dk / VEC;
+        for (int idx = threadIdx.x; idx < ng * MX_KEYS * pieces; idx += MX_THREADS) {
+          const int p = idx % pieces, kk = (idx / pieces) % MX_KEYS, gl = idx / (pieces * MX_KEYS);
+          const bool ok = kk < nk;
+          cp_async16((uint32_t)__cvta_generic_to_shared(kst + ((size_t)gl * MX_KEYS + kk) * KP + p * VEC),
+                     kb + ((int64_t)(g0 + gl) * Tcap + j0 + (ok ? kk : 0)) * dk + p * VEC, ok);
+        }
+        cp_async_commit();
+        cp_async_wait<0>();
+      } else {
+        for (int idx = threadIdx.x; idx < ng * MX_KEYS * dk; idx += MX_THREADS) {
+          const int i = idx % dk, kk = (idx / dk) % MX_KEYS, gl = idx / (dk * MX_KEYS);
+          kst[((size_t)gl * MX_KEYS + kk) * KP + i] = kk < nk ? kb[((int64_t)(g0 + gl) * Tcap + j0 + kk) * dk + i] : Tr<T>::from_f(0.f);
+        }
+      }
+      __syncthreads();
+      const int blocks = (per + MX_HEADS - 1) / MX_HEADS;
+      for (int it = warp; it < ng * blocks; it += nw) {
+        const int gl = it / blocks, h0 = (it % blocks) * MX_HEADS;   // heads h0 .. of the key head, some of which may not exist
+        const T* kr = kst + ((size_t)gl * MX_KEYS + lane) * KP;
+        const float* qr[MX_HEADS];
+        float d[MX_HEADS];
+#pragma unroll
+        for (int k = 0; k < MX_HEADS; ++k) {
+          qr[k] = qs + (size_t)((g0 + gl) * per + min(h0 + k, per - 1)) * dk;
+          d[k] = 0.f;
+        }
+        for (int i = 0; i < dk; i += VEC) {
+          float kv[VEC];
+          if constexpr (VEC > 1) {
+            const uint4 u = *reinterpret_cast<const uint4*>(kr + i);
+            const T* e = reinterpret_cast<const T*>(&u);
+#pragma unroll
+            for (int k = 0; k < VEC; ++k) kv[k] = Tr<T>::to_f(e[k]);
+          } else {
+            kv[0] = Tr<T>::to_f(kr[i]);
+          }
+#pragma unroll
+          for (int k = 0; k < MX_HEADS; ++k)
+#pragma unroll
+            for (int x = 0; x < VEC; ++x) d[k] = fmaf(qr[k][i + x], kv[x], d[k]);
+        }
+#pragma unroll
+        for (int k = 0; k < MX_HEADS; ++k)
+          if (h0 + k < per) raw[((g0 + gl) * per + h0 + k) * MX_KEYS + lane] = d[k];
+      }
+    }
+    __syncthreads();
+    for (int h = warp; h < H; h += nw) {                             // mix and soften: lane = key
+      float s = 0.f;
+      for (int g = 0; g < H; ++g) s = fmaf(tk[h * H + g], raw[g * MX_KEYS + lane], s);
+      if (lane >= nk) s = -INFINITY;
+      const float mo = m_s[h], mn = fmaxf(mo, warp_max(s));          // finite: every chunk holds a visible key
+      const float p = lane < nk ? expf(s - mn) : 0.f, sum = warp_sum(p), corr = expf(mo - mn);
+      pr[h * MX_KEYS + lane] = p;
+      __syncwarp();
+      if (lane == 0) { m_s[h] = mn; l_s[h] = l_s[h] * corr + sum; c_s[h] = corr; }
+    }
+    __syncthreads();
+    const int vpieces = dv / VEC;
+    for (int idx = threadIdx.x; idx < H * vpieces; idx += MX_THREADS) {
+      const int h = idx / vpieces, p = idx % vpieces;
+      float a[VEC];
+      const float corr = c_s[h];
+#pragma unroll
+      for (int x = 0; x < VEC; ++x) a[x] = acc[h * dv + p * VEC + x] * corr;
+      const T* vr = vb + ((int64_t)(h / per) * Tcap + j0) * dv + p * VEC;
+#pragma unroll 8
+      for (int kk = 0; kk < nk; ++kk) {
+        const float w = pr[h * MX_KEYS + kk];
+        if constexpr (VEC > 1) {
+          const uint4 u = *reinterpret_cast<const uint4*>(vr + (int64_t)kk * dv);
+          const T* e = reinterpret_cast<const T*>(&u);
+#pragma unroll
+          for (int x = 0; x < VEC; ++x) a[x] = fmaf(w, Tr<T>::to_f(e[x]), a[x]);
+        } else {
+          a[0] = fmaf(w, Tr<T>::to_f(vr[(int64_t)kk * dv]), a[0]);
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < VEC; ++x) acc[h * dv + p * VEC + x] = a[x];
+    }
+  }
+  __syncthreads();
+  if (whole) {
+    for (int i = threadIdx.x; i < H * dv; i += MX_THREADS) out[t * ld_out + i] = Tr<T>::from_f(acc[i] / l_s[i / dv]);
+    return;
+  }
+  for (int h = threadIdx.x; h < H; h += MX_THREADS) {
+    float* ms = part_ms + ((t * H + h) * gridDim.x + blockIdx.x) * 2;
+    ms[0] = m_s[h] * LOG2E;                                          // a share without keys leaves (-inf, 0)
+    ms[1] = l_s[h];
+  }
+  if (c_lo < c_hi)
+    for (int i = threadIdx.x; i < H * dv; i += MX_THREADS)
+      part_o[((t * H + i / dv) * gridDim.x + blockIdx.x) * dv + i % dv] = acc[i];
+}
+
+// ---- prompts on the tensor cores ---------------------------------------------------------------------------------------------
+__device__ __forceinline__ uint32_t to_tf32(float x) {
+  uint32_t r;
+  asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x));
+  return r;
+}
+__device__ __forceinline__ void mma1688_tf32(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+constexpr int MT_MAX_WARPS = 16;
+
+// shared floats: one head's raw scores (QB queries x KT keys; the paddings keep fragment accesses free of bank conflicts)
+constexpr int mt_pitch(int kt) { return kt + 8; }
+constexpr int mt_head(int hb, int kt) { return 16 / hb * mt_pitch(kt) + 8; }
+static size_t mt_smem(int H, int G, int dk, int dv, int hb, int kt) {
+  const int hp = (H + 7) / 8 * 8, mb = hb;
+  return (size_t)G * kt * (dk + dv) * 2 + (size_t)hp * mt_head(hb, kt) * 4 + (size_t)mb * 16 * (hp + 4) * 4;
+}
+
+// CTA = QB = 16 / HB consecutive queries (tile blockIdx.x) of entry blockIdx.y, all H heads; warp w owns the heads w HB .. w HB + HB-1
+// (HB = 2: two heads of one key/value head fill the 16 rows of a fragment with 8 queries each).  Per chunk of KT keys:
+//   raw scores of the warp's heads -> shared; all heads of 8 key positions at a time mixed in place by any warp; mixed scores of
+//   the warp's heads -> window, online softmax in registers (base-2 units, opened by the sink), O += P V.
+// Keys and values of all key/value heads sit in one buffer each: values arrive while scores are formed, the next keys while
+// scores are mixed and values multiplied.
+template <typename T, int DK, int DV, int HB, int KT>
+__global__ void __launch_bounds__(MT_MAX_WARPS * 32, 1)
+mix_attn_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc, const T* __restrict__ vc, int64_t Tcap,
+                     const int32_t* __restrict__ cu, const int32_t* __restrict__ rows, const int32_t* __restrict__ t_pos,
+                     const float* __restrict__ talk, const float* __restrict__ sink, int window, T* __restrict__ out, int64_t ld_out,
+                     int H, int G) {
+  constexpr int QB = 16 / HB, PITCH = mt_pitch(KT), HS = mt_head(HB, KT), MB = HB;
+  constexpr int KROW = DK * 2, VROW = DV * 2, KCH = DK / 8, VCH = DV / 8;
+  extern __shared__ __align__(128) uint8_t mt_sm[];
+  const int e = blockIdx.y;
+  const int t_first = cu[e], n_e = cu[e + 1] - t_first;
+  const int q0 = blockIdx.x * QB;
+  if (q0 >= n_e) return;                                             // the same for every thread of the CTA
+  const int NT = blockDim.x, NW = NT >> 5;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, quad_row = lane >> 2, qc = lane & 3;
+  const int HP = (H + 7) / 8 * 8, TP = HP + 4;
+  const int per = H / G;
+  const int h0 = warp * HB, h1 = HB == 2 ? h0 + 1 : h0;              // heads of the fragment's rows 0-7 and 8-15
+  const int g = h0 / per;
+  const int l0 = q0 + quad_row, l1 = HB == 2 ? l0 : l0 + 8;          // the rows' queries (offsets in the entry)
+  const int lc0 = min(l0, n_e - 1), lc1 = min(l1, n_e - 1);          // rows past the end compute a valid row, not stored
+  const int p_first = t_pos[t_first];                                // positions of an entry's tokens are consecutive
+  const int pos0 = p_first + lc0, pos1 = p_first + lc1;
+  const int kend = p_first + min(n_e, q0 + QB);                      // keys any row of this CTA may see
+  const int first = window > 0 ? p_first + q0 - window + 1 : 0;      // the first key the CTA's first row sees
+  const int tile_lo = first > 0 ? first / KT : 0, tile_hi = (kend + KT - 1) / KT;
+  const uint32_t ks = (uint32_t)__cvta_generic_to_shared(mt_sm), vs = ks + G * KT * KROW;
+  float* raw = reinterpret_cast<float*>(mt_sm + (size_t)G * KT * (KROW + VROW));      // [HP][HS]
+  float* tks = raw + HP * HS;                                        // [MB * 16][TP], zeros outside H x H
+  for (int i = threadIdx.x; i < (HP - H) * HS; i += NT) raw[H * HS + i] = 0.f;        // padded heads meet zero weights: keep them finite
+  for (int i = threadIdx.x; i < MB * 16 * TP; i += NT) {
+    const int a = i / TP, b = i % TP;
+    tks[i] = (a < H && b < H) ? talk[a * H + b] : 0.f;
+  }
+
+  uint32_t qf[DK / 16][4];
+  {
+    const float* p0 = q + ((int64_t)(t_first + lc0) * H + h0) * DK;
+    const float* p1 = q + ((int64_t)(t_first + lc1) * H + h1) * DK;
+#pragma unroll
+    for (int s = 0; s < DK / 16; ++s) {
+      const float2 a0 = *reinterpret_cast<const float2*>(p0 + s * 16 + 2 * qc), a1 = *reinterpret_cast<const float2*>(p1 + s * 16 + 2 * qc);
+      const float2 b0 = *reinterpret_cast<const float2*>(p0 + s * 16 + 8 + 2 * qc), b1 = *reinterpret_cast<const float2*>(p1 + s * 16 + 8 + 2 * qc);
+      qf[s][0] = pack2<T>(a0.x, a0.y);
+      qf[s][1] = pack2<T>(a1.x, a1.y);
+      qf[s][2] = pack2<T>(b0.x, b0.y);
+      qf[s][3] = pack2<T>(b1.x, b1.y);
+    }
+  }
+  const int64_t row = rows[e];
+  auto load_keys = [&](int tile) {
+    const int key0 = tile * KT;
+    for (int idx = threadIdx.x; idx < G * KT * KCH; idx += NT) {
+      const int ch = idx % KCH, key = (idx / KCH) % KT, gg = idx / (KCH * KT);
+      const bool ok = key0 + key < kend;
+      cp_async16(ks + (uint32_t)((gg * KT + key) * KROW + ((ch ^ (key & 7)) << 4)),
+                 kc + ((row * G + gg) * Tcap + key0 + (ok ? key : 0)) * DK + ch * 8, ok);
+    }
+  };
+  auto load_values = [&](int tile) {
+    const int key0 = tile * KT;
+    for (int idx = threadIdx.x; idx < G * KT * VCH; idx += NT) {
+      const int ch = idx % VCH, key = (idx / VCH) % KT, gg = idx / (VCH * KT);
+      const bool ok = key0 + key < kend;
+      cp_async16(vs + (uint32_t)((gg * KT + key) * VROW + ((ch ^ (key & 7)) << 4)),
+                 vc + ((row * G + gg) * Tcap + key0 + (ok ? key : 0)) * DV + ch * 8, ok);
+    }
+  };
+
+  float o[DV / 8][4];
+#pragma unroll
+  for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  // the sink opens the softmax: it is the running maximum, and its own term (one) sits in the sum of one thread of the quad
+  float m0 = sink ? sink[h0] * LOG2E : -INFINITY, m1 = sink ? sink[h1] * LOG2E : -INFINITY;
+  float s0 = (sink && qc == 0) ? 1.f : 0.f, s1 = s0;
+  const int wnd = window > 0 ? window : 0x7fffffff;
+  const int mat = lane >> 3, r8 = lane & 7;
+  const uint32_t kg = ks + g * KT * KROW, vg = vs + g * KT * VROW;
+
+  load_keys(tile_lo);
+  cp_async_commit();
+  for (int it = tile_lo; it < tile_hi; ++it) {
+    cp_async_wait<0>();                                              // this chunk's keys
+    __syncthreads();                                                 // ... of every thread; the last chunk's values and scores are used up
+    load_values(it);
+    cp_async_commit();
+    float sc[KT / 8][4];
+#pragma unroll
+    for (int nt = 0; nt < KT / 8; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
+#pragma unroll
+    for (int np = 0; np < KT / 16; ++np) {
+      const int key = 16 * np + r8 + 8 * (mat >> 1);
+#pragma unroll
+      for (int s = 0; s < DK / 16; ++s) {
+        const int ch = 2 * s + (mat & 1);
+        uint32_t bf[4];
+        ldsm_x4(kg + (uint32_t)(key * KROW + ((ch ^ (key & 7)) << 4)), bf);
+        mma16816<T>(sc[2 * np], qf[s], bf[0], bf[1]);
+        mma16816<T>(sc[2 * np + 1], qf[s], bf[2], bf[3]);
+      }
+    }
+    float* raw0 = raw + h0 * HS + quad_row * PITCH + 2 * qc;         // this thread's two fragment rows
+    float* raw1 = HB == 2 ? raw0 + HS : raw0 + 8 * PITCH;
+#pragma unroll
+    for (int nt = 0; nt < KT / 8; ++nt) {
+      *reinterpret_cast<float2*>(raw0 + 8 * nt) = make_float2(sc[nt][0], sc[nt][1]);
+      *reinterpret_cast<float2*>(raw1 + 8 * nt) = make_float2(sc[nt][2], sc[nt][3]);
+    }
+    __syncthreads();                                                 // raw scores of all heads; the keys are used up
+    if (it + 1 < tile_hi) load_keys(it + 1);
+    cp_async_commit();
+    // mixed = talk x raw, 8 key positions of one query at a time (columns), heads as rows and as the summed index
+    for (int nt = warp; nt < QB * KT / 8; nt += NW) {
+      float* base = raw + (nt / (KT / 8)) * PITCH + (nt % (KT / 8)) * 8;
+      float c[MB][4];
+#pragma unroll
+      for (int mb = 0; mb < MB; ++mb) c[mb][0] = c[mb][1] = c[mb][2] = c[mb][3] = 0.f;
+#pragma unroll
+      for (int s = 0; s < 2 * MB; ++s) {
+        if (s * 8 < HP) {
+          const float x0 = base[(s * 8 + qc) * HS + quad_row], x1 = base[(s * 8 + 4 + qc) * HS + quad_row];
+          const uint32_t hi0 = to_tf32(x0), hi1 = to_tf32(x1);       // x = hi + lo to 22 bits; the weights are exact in tf32
+          const uint32_t lo0 = to_tf32(x0 - __uint_as_float(hi0)), lo1 = to_tf32(x1 - __uint_as_float(hi1));
+#pragma unroll
+          for (int mb = 0; mb < MB; ++mb) {
+            const float* tr = tks + (mb * 16 + quad_row) * TP + s * 8 + qc;
+            const uint32_t a[4] = {__float_as_uint(tr[0]), __float_as_uint(tr[8 * TP]), __float_as_uint(tr[4]), __float_as_uint(tr[8 * TP + 4])};
+            mma1688_tf32(c[mb], a, lo0, lo1);
+            mma1688_tf32(c[mb], a, hi0, hi1);
+          }
+        }
+      }
+      __syncwarp();                                                  // every lane has read these positions
+#pragma unroll
+      for (int mb = 0; mb < MB; ++mb) {
+        const int ha = mb * 16 + quad_row, hb = ha + 8;
+        if (ha < H) *reinterpret_cast<float2*>(base + ha * HS + 2 * qc) = make_float2(c[mb][0], c[mb][1]);
+        if (hb < H) *reinterpret_cast<float2*>(base + hb * HS + 2 * qc) = make_float2(c[mb][2], c[mb][3]);
+      }
+    }
+    cp_async_wait<1>();                                              // the values (the next keys may still be on their way)
+    __syncthreads();                                                 // ... of every thread, and the mixed scores
+    float t0 = -INFINITY, t1 = -INFINITY;
+#pragma unroll
+    for (int nt = 0; nt < KT / 8; ++nt) {
+      const float2 a = *reinterpret_cast<const float2*>(raw0 + 8 * nt), b = *reinterpret_cast<const float2*>(raw1 + 8 * nt);
+      const int kcol = it * KT + 8 * nt + 2 * qc;
+      const int d0 = pos0 - kcol, d1 = pos1 - kcol;
+      sc[nt][0] = (d0 >= 0 && d0 < wnd) ? a.x * LOG2E : -INFINITY;
+      sc[nt][1] = (d0 >= 1 && d0 <= wnd) ? a.y * LOG2E : -INFINITY;
+      sc[nt][2] = (d1 >= 0 && d1 < wnd) ? b.x * LOG2E : -INFINITY;
+      sc[nt][3] = (d1 >= 1 && d1 <= wnd) ? b.y * LOG2E : -INFINITY;
+      t0 = fmaxf(t0, fmaxf(sc[nt][0], sc[nt][1]));
+      t1 = fmaxf(t1, fmaxf(sc[nt][2], sc[nt][3]));
+    }
+    t0 = fmaxf(t0, __shfl_xor_sync(0xffffffffu, t0, 1)); t0 = fmaxf(t0, __shfl_xor_sync(0xffffffffu, t0, 2));
+    t1 = fmaxf(t1, __shfl_xor_sync(0xffffffffu, t1, 1)); t1 = fmaxf(t1, __shfl_xor_sync(0xffffffffu, t1, 2));
+    const float keep0 = fmaxf(m0, t0), keep1 = fmaxf(m1, t1);
+    // nothing seen yet (the row's window begins later and there is no sink): exponentials against 0
+    const float mn0 = keep0 == -INFINITY ? 0.f : keep0, mn1 = keep1 == -INFINITY ? 0.f : keep1;
+    const float corr0 = exp2f(m0 - mn0), corr1 = exp2f(m1 - mn1);
+    m0 = keep0; m1 = keep1;
+    float ps0 = 0.f, ps1 = 0.f;
+#pragma unroll
+    for (int nt = 0; nt < KT / 8; ++nt) {
+      sc[nt][0] = exp2f(sc[nt][0] - mn0); sc[nt][1] = exp2f(sc[nt][1] - mn0);
+      sc[nt][2] = exp2f(sc[nt][2] - mn1); sc[nt][3] = exp2f(sc[nt][3] - mn1);
+      ps0 += sc[nt][0] + sc[nt][1];
+      ps1 += sc[nt][2] + sc[nt][3];
+    }
+    s0 = s0 * corr0 + ps0;
+    s1 = s1 * corr1 + ps1;
+#pragma unroll
+    for (int j = 0; j < DV / 8; ++j) { o[j][0] *= corr0; o[j][1] *= corr0; o[j][2] *= corr1; o[j][3] *= corr1; }
+#pragma unroll
+    for (int kk = 0; kk < KT / 16; ++kk) {
+      uint32_t pf[4];
+      pf[0] = pack2<T>(sc[2 * kk][0], sc[2 * kk][1]);
+      pf[1] = pack2<T>(sc[2 * kk][2], sc[2 * kk][3]);
+      pf[2] = pack2<T>(sc[2 * kk + 1][0], sc[2 * kk + 1][1]);
+      pf[3] = pack2<T>(sc[2 * kk + 1][2], sc[2 * kk + 1][3]);
+      const int key = 16 * kk + r8 + 8 * (mat & 1);
+#pragma unroll
+      for (int jp = 0; jp < DV / 16; ++jp) {
+        const int ch = 2 * jp + (mat >> 1);
+        uint32_t bf[4];
+        ldsm_x4_trans(vg + (uint32_t)(key * VROW + ((ch ^ (key & 7)) << 4)), bf);
+        mma16816<T>(o[2 * jp], pf, bf[0], bf[1]);
+        mma16816<T>(o[2 * jp + 1], pf, bf[2], bf[3]);
+      }
+    }
+  }
+  cp_async_wait<0>();
+  s0 += __shfl_xor_sync(0xffffffffu, s0, 1); s0 += __shfl_xor_sync(0xffffffffu, s0, 2);
+  s1 += __shfl_xor_sync(0xffffffffu, s1, 1); s1 += __shfl_xor_sync(0xffffffffu, s1, 2);
+  const float inv0 = 1.f / s0, inv1 = 1.f / s1;
+  T* o0 = out + (int64_t)(t_first + lc0) * ld_out + (int64_t)h0 * DV;
+  T* o1 = out + (int64_t)(t_first + lc1) * ld_out + (int64_t)h1 * DV;
+#pragma unroll
+  for (int j = 0; j < DV / 8; ++j) {
+    const int c = 8 * j + 2 * qc;
+    if (l0 < n_e) *reinterpret_cast<uint32_t*>(o0 + c) = pack2<T>(o[j][0] * inv0, o[j][1] * inv0);
+    if (l1 < n_e) *reinterpret_cast<uint32_t*>(o1 + c) = pack2<T>(o[j][2] * inv1, o[j][3] * inv1);
+  }
+}
+
+template <typename T, int DK, int DV, int HB, int KT>
+static int mix_attn_tile_launch(const float* q, const void* kc, const void* vc, int64_t Tcap, const int32_t* cu, const int32_t* rows,
+                                const int32_t* t_pos, const float* talk, const float* sink, int window, void* out, int64_t ld_out, int nb,
+                                int max_n, int H, int G, size_t smem, cudaStream_t st) {
+  auto kern = mix_attn_tile_kernel<T, DK, DV, HB, KT>;
+  static bool attr = false;
+  if (!attr) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, MX_SMEM_MAX);
+    if (e != cudaSuccess) return cuda_fail(e, "cudaFuncSetAttribute(mix_attn_tile_kernel)");
+    attr = true;
+  }
+  constexpr int QB = 16 / HB;
+  dim3 grid((unsigned)((max_n + QB - 1) / QB), (unsigned)nb);
+  kern<<<grid, (unsigned)((H + HB - 1) / HB * 32), smem, st>>>(q, (const T*)kc, (const T*)vc, Tcap, cu, rows, t_pos, talk, sink, window,
+                                                                (T*)out, ld_out, H, G);
+  B200P_LAUNCH_CHECK("mix_attn_tile_kernel");
+  return B200P_OK;
+}
+
+// heads per warp (1 or 2) and keys per chunk (32 or 16) of the tile kernel; false when it does not take these sizes
+static bool mix_attn_tile_plan(int H, int G, int dk, int dv, int dtype, int* hb, int* kt) {
+  if ((dtype != B200P_F16 && dtype != B200P_BF16) || (dk != 64 && dk != 128) || (dv != 64 && dv != 128)) return false;
+  if (H <= MT_MAX_WARPS) *hb = 1;
+  else if (H <= 2 * MT_MAX_WARPS && (H / G) % 2 == 0) *hb = 2;
+  else return false;
+  for (*kt = 32; *kt >= 16; *kt /= 2)
+    if (mt_smem(H, G, dk, dv, *hb, *kt) <= (size_t)MX_SMEM_MAX) return true;
+  return false;
+}
+
+template <typename T>
+static int mix_attn_tiles(const float* q, const void* kc, const void* vc, int64_t Tcap, const int32_t* cu, const int32_t* rows,
+                          const int32_t* t_pos, const float* talk, const float* sink, int window, void* out, int64_t ld_out, int nb,
+                          int max_n, int H, int G, int dk, int dv, int hb, int kt, cudaStream_t st) {
+  const size_t smem = mt_smem(H, G, dk, dv, hb, kt);
+#define MT_CASE(DK_, DV_, HB_, KT_)                                                                                               \
+  if (dk == DK_ && dv == DV_ && hb == HB_ && kt == KT_)                                                                           \
+    return mix_attn_tile_launch<T, DK_, DV_, HB_, KT_>(q, kc, vc, Tcap, cu, rows, t_pos, talk, sink, window, out, ld_out, nb, max_n, H, G, smem, st)
+#define MT_SIZES(DK_, DV_) MT_CASE(DK_, DV_, 1, 32); MT_CASE(DK_, DV_, 1, 16); MT_CASE(DK_, DV_, 2, 32); MT_CASE(DK_, DV_, 2, 16)
+  MT_SIZES(64, 64);
+  MT_SIZES(64, 128);
+  MT_SIZES(128, 64);
+  MT_SIZES(128, 128);
+#undef MT_SIZES
+#undef MT_CASE
+  set_error("mixed-score tile attention: unsupported sizes");
+  return B200P_ERR_ARG;
+}
+
+constexpr int MIX_ATTN_TILES_MIN_TOKENS = 4;   // shorter portions (and decode steps) take the per-token kernel
+
+template <typename T, int VEC>
+static int mix_attn_token(const float* q, const void* kc, const void* vc, int64_t Tcap, const int32_t* t_row, const int32_t* t_pos,
+                          const float* talk, const float* sink, int64_t window, void* out, int64_t ld_out, int64_t M, int H, int G, int dk,
+                          int dv, bool split, float* ws, size_t ws_bytes, cudaStream_t st) {
+  const int KP = VEC > 1 ? dk + VEC : dk + 1;
+  const size_t per_kv = (size_t)MX_KEYS * KP * sizeof(T), rest = ((size_t)H * (dk + dv + H + 2 * MX_KEYS + 3)) * sizeof(float) + 16;
+  B200P_REQUIRE(rest + per_kv <= (size_t)MX_SMEM_MAX, B200P_ERR_ARG, "%d heads of %d / %d values do not fit the per-token kernel", H, dk, dv);
+  size_t room = MX_SMEM_MAX - rest;
+  if (room > 48 * 1024) room = per_kv > 48 * 1024 ? per_kv : 48 * 1024;          // leave room for several CTAs per SM
+  int kv_block = (int)(room / per_kv);
+  if (kv_block > G) kv_block = G;
+  const size_t smem = rest + kv_block * per_kv;
+  auto kern = mix_attn_kernel<T, VEC>;
+  static size_t attr_smem = 48 * 1024;
+  if (smem > attr_smem) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return cuda_fail(e, "cudaFuncSetAttribute(mix_attn_kernel)");
+    attr_smem = smem;
+  }
+  int splits = 1;
+  const size_t per_split = (size_t)M * H * (dv + 2) * sizeof(float);
+  if (split) {
+    splits = (int)((4 * 148 + M - 1) / M);
+    splits = splits < 1 ? 1 : splits > MX_MAX_SPLITS ? MX_MAX_SPLITS : splits;
+    if ((size_t)splits * per_split > ws_bytes) splits = (int)(ws_bytes / per_split);
+  }
+  B200P_REQUIRE(M < 65536, B200P_ERR_ARG, "at most 65535 tokens per call");
+  if (splits <= 1) {
+    kern<<<dim3(1, (unsigned)M), MX_THREADS, smem, st>>>(q, (const T*)kc, (const T*)vc, Tcap, t_row, t_pos, talk, sink, window, (T*)out, ld_out,
+                                                          H, G, dk, dv, nullptr, nullptr, kv_block);
+    B200P_LAUNCH_CHECK("mix_attn_kernel");
+    return B200P_OK;
+  }
+  float* part_o = ws;
+  float* part_ms = ws + (size_t)M * H * splits * dv;
+  kern<<<dim3((unsigned)splits, (unsigned)M), MX_THREADS, smem, st>>>(q, (const T*)kc, (const T*)vc, Tcap, t_row, t_pos, talk, sink, window,
+                                                                       (T*)out, ld_out, H, G, dk, dv, part_o, part_ms, kv_block);
+  B200P_LAUNCH_CHECK("mix_attn_kernel");
+  attn_merge_kernel<T><<<dim3((unsigned)M, (unsigned)H), dv >= 128 ? 128 : 64, 0, st>>>(part_o, part_ms, nullptr, sink, (T*)out, ld_out, 1.f, H,
+                                                                                         dv, splits, nullptr, 0);
+  B200P_LAUNCH_CHECK("attn_merge_kernel");
+  return B200P_OK;
+}
+
+}  // namespace b200p
+
+using namespace b200p;
+
+extern "C" int b200p_mix_attn_prep(const float* proj, int64_t ldp, int64_t col_q, int64_t col_k, int64_t col_v, const float* bias,
+                                   const float* wq, const float* wk, float eps, const float* rates, int n_rot, float mag, int pairs,
+                                   float scale, float* q_out, void* kcache, void* vcache, int64_t Tcap, const int32_t* t_row,
+                                   const int32_t* t_pos, int64_t M, int H, int G, int dk, int dv, int dtype, void* stream) {
+  B200P_REQUIRE(proj && q_out && kcache && vcache && t_row && t_pos, B200P_ERR_ARG, "null pointer");
+  B200P_REQUIRE(H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0, B200P_ERR_ARG, "bad head geometry");
+  B200P_REQUIRE(n_rot >= 0 && 2 * n_rot <= dk && n_rot <= 4096 && (n_rot == 0 || rates), B200P_ERR_ARG, "at most dk dimensions are rotated");
+  B200P_REQUIRE(!(pairs && n_rot) || dk % 2 == 0, B200P_ERR_ARG, "pairwise rotation needs heads of an even size");
+  if (M == 0) return B200P_OK;
+  const bool vec = !pairs && dk % 4 == 0 && n_rot % 4 == 0 && ldp % 4 == 0 && col_q % 4 == 0 && col_k % 4 == 0 && aligned(proj, 16) &&
+                   aligned(bias, 16) && aligned(q_out, 16);
+  const size_t smem = 2 * (size_t)n_rot * sizeof(float);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (vec) {
+    B200P_DISPATCH_DTYPE(dtype, T, (mix_attn_prep_kernel<T, 4><<<(unsigned)M, 256, smem, st>>>(
+        proj, ldp, col_q, col_k, col_v, bias, wq, wk, eps, rates, n_rot, mag, pairs, scale, q_out, (T*)kcache, (T*)vcache, Tcap, t_row, t_pos,
+        H, G, dk, dv)));
+  } else {
+    B200P_DISPATCH_DTYPE(dtype, T, (mix_attn_prep_kernel<T, 1><<<(unsigned)M, 256, smem, st>>>(
+        proj, ldp, col_q, col_k, col_v, bias, wq, wk, eps, rates, n_rot, mag, pairs, scale, q_out, (T*)kcache, (T*)vcache, Tcap, t_row, t_pos,
+        H, G, dk, dv)));
+  }
+  B200P_LAUNCH_CHECK("mix_attn_prep_kernel");
+  return B200P_OK;
+}
+
+extern "C" size_t b200p_mix_attn_workspace_bytes(int64_t nb, int H, int dv) {
+  return (size_t)nb * H * MX_MAX_SPLITS * (dv + 2) * sizeof(float);
+}
+
+extern "C" int b200p_mix_attn_tiles_supported(int H, int G, int dk, int dv, int dtype) {
+  int hb, kt;
+  return H > 0 && G > 0 && H % G == 0 && mix_attn_tile_plan(H, G, dk, dv, dtype, &hb, &kt) ? hb * 100 + kt : 0;
+}
+
+extern "C" int b200p_mix_attn(const float* q, const void* kcache, const void* vcache, int64_t Tcap, const int32_t* t_row,
+                              const int32_t* t_pos, const int32_t* cu, const int32_t* rows, int nb, int max_n, const float* talk,
+                              const float* sink, int64_t window, void* out, int64_t ld_out, int64_t M, int H, int G, int dk, int dv,
+                              int dtype, void* workspace, size_t workspace_bytes, void* stream) {
+  B200P_REQUIRE(q && kcache && vcache && t_row && t_pos && talk && out, B200P_ERR_ARG, "null pointer");
+  B200P_REQUIRE(H > 0 && G > 0 && H % G == 0 && dk > 0 && dv > 0, B200P_ERR_ARG, "bad head geometry");
+  B200P_REQUIRE(window >= 0 && window < 0x7fffffff, B200P_ERR_ARG, "bad window");
+  B200P_REQUIRE(ld_out >= (int64_t)H * dv, B200P_ERR_ARG, "output rows are shorter than the heads");
+  if (M == 0) return B200P_OK;
+  cudaStream_t st = (cudaStream_t)stream;
+  int hb = 0, kt = 0;
+  if (cu && rows && nb > 0 && nb < 65536 && max_n >= MIX_ATTN_TILES_MIN_TOKENS && ld_out % 2 == 0 && aligned(kcache, 16) &&
+      aligned(vcache, 16) && aligned(out, 4) && aligned(q, 8) && mix_attn_tile_plan(H, G, dk, dv, dtype, &hb, &kt)) {
+    return dtype == B200P_F16
+        ? mix_attn_tiles<__half>(q, kcache, vcache, Tcap, cu, rows, t_pos, talk, sink, (int)window, out, ld_out, nb, max_n, H, G, dk, dv, hb, kt, st)
+        : mix_attn_tiles<__nv_bfloat16>(q, kcache, vcache, Tcap, cu, rows, t_pos, talk, sink, (int)window, out, ld_out, nb, max_n, H, G, dk, dv, hb,
+                                        kt, st);
+  }
+  // 16-bit decode steps (one token per entry) split their keys over CTAs, given room for the partial sums
+  const bool split = max_n == 1 && dtype != B200P_F32 && workspace && aligned(workspace, 16);
+  const int vec = dtype == B200P_F32 ? 4 : 8;
+  const bool whole = dk % vec == 0 && dv % vec == 0 && aligned(kcache, 16) && aligned(vcache, 16);
+#define MX_CASE(T, V_) \
+  mix_attn_token<T, V_>(q, kcache, vcache, Tcap, t_row, t_pos, talk, sink, window, out, ld_out, M, H, G, dk, dv, split, (float*)workspace, workspace_bytes, st)
+  switch (dtype) {
+    case B200P_F32: return whole ? MX_CASE(float, 4) : MX_CASE(float, 1);
+    case B200P_F16: return whole ? MX_CASE(__half, 8) : MX_CASE(__half, 1);
+    case B200P_BF16: return whole ? MX_CASE(__nv_bfloat16, 8) : MX_CASE(__nv_bfloat16, 1);
+    default: set_error("bad dtype %d", dtype); return B200P_ERR_ARG;
+  }
+#undef MX_CASE
+}

@@ -1,7 +1,8 @@
 // Routed mixture of experts over a packed token batch:
 //   moe_route_kernel    fp32 router logits (+ bias) -> the `top` largest per token and the softmax over those alone   (per token)
 //   moe_route_sigmoid_kernel  scores = sigmoid(logits); experts picked by score + correction inside the best expert groups;
-//                       weights = the picked experts' scores over their sum, times a scale                              (per token)
+//                       weights = the picked experts' scores over their sum, times a scale; or the scores as they are, of
+//                       sigmoids or of a softmax over all experts                                                       (per token)
 //   moe_plan_kernel     tokens counted per expert, segment offsets, a slot for every (token, choice)                 (one CTA)
 //   moe_gather_kernel   activation rows copied into slot order, so that an expert's rows are contiguous              (per slot)
 //   moe_combine_kernel  y[t] = gate[t] shared[t] + sum_k weight[t, k] * expert_out[slot(t, k)], in the order of the choices   (per token)
@@ -59,7 +60,7 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ldl, 
 // largest picking scores win, ties to the smaller index; weights w_k = s_k / (sum of the picked s + 1e-20) * scale.
 __global__ void moe_route_sigmoid_kernel(const float* __restrict__ logits, int64_t ldl, const float* __restrict__ correction,
                                          int32_t* __restrict__ ids, float* __restrict__ wts, int64_t M, int E, int top, int count,
-                                         int keep, float scale, int renorm) {
+                                         int keep, float scale, int renorm, int softmax) {
   extern __shared__ float mr_sm[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int64_t t = (int64_t)blockIdx.x * (blockDim.x >> 5) + warp;
@@ -67,10 +68,24 @@ __global__ void moe_route_sigmoid_kernel(const float* __restrict__ logits, int64
   float* sc = mr_sm + (size_t)warp * (2 * E + count);     // scores
   float* pick = sc + E;                                    // picking scores, -inf once masked or taken
   float* gs = pick + E;                                    // group scores
-  for (int e = lane; e < E; e += 32) {
-    const float s = 1.f / (1.f + expf(-logits[t * ldl + e]));
-    sc[e] = s;
-    pick[e] = s + (correction ? correction[e] : 0.f);
+  if (softmax) {                                           // scores = softmax over ALL experts; picked by the logits themselves
+    float top1 = -INFINITY, sum = 0.f;
+    for (int e = lane; e < E; e += 32) top1 = fmaxf(top1, logits[t * ldl + e]);
+    top1 = warp_max(top1);
+    for (int e = lane; e < E; e += 32) {
+      const float z = logits[t * ldl + e], p = expf(z - top1);
+      sum += p;
+      sc[e] = p;
+      pick[e] = z;
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) sc[e] /= sum;
+  } else {
+    for (int e = lane; e < E; e += 32) {
+      const float s = 1.f / (1.f + expf(-logits[t * ldl + e]));
+      sc[e] = s;
+      pick[e] = s + (correction ? correction[e] : 0.f);
+    }
   }
   __syncwarp();
   if (count > 1 && keep < count) {
@@ -248,7 +263,7 @@ extern "C" int b200p_moe_route_sigmoid(const float* logits, int64_t ldl, const f
     if (e != cudaSuccess) return cuda_fail(e, "cudaFuncSetAttribute(moe_route_sigmoid_kernel)");
   }
   moe_route_sigmoid_kernel<<<(unsigned)((M + warps - 1) / warps), warps * 32, smem, st>>>(logits, ldl, correction, ids, wts, M, E, top,
-                                                                                           count, keep, scale, 1);
+                                                                                           count, keep, scale, 1, 0);
   B200P_LAUNCH_CHECK("moe_route_sigmoid_kernel");
   moe_plan_kernel<<<1, 1024, 2 * E * sizeof(int32_t), st>>>(ids, seg, slot_of, token_of, M * top, E, top);
   B200P_LAUNCH_CHECK("moe_plan_kernel");
@@ -256,7 +271,7 @@ extern "C" int b200p_moe_route_sigmoid(const float* logits, int64_t ldl, const f
 }
 
 extern "C" int b200p_moe_route_scores(const float* logits, int64_t ldl, int32_t* ids, float* wts, int32_t* seg, int32_t* slot_of,
-                                      int32_t* token_of, int64_t M, int E, int top, void* stream) {
+                                      int32_t* token_of, int64_t M, int E, int top, int softmax, void* stream) {
   B200P_REQUIRE(logits && ids && wts && seg && slot_of && token_of, B200P_ERR_ARG, "null pointer");
   B200P_REQUIRE(E > 0 && E <= 32 * MOE_MAX_PER_LANE && top > 0 && top <= E && top <= MOE_MAX_TOP, B200P_ERR_ARG,
                 "experts in [1, %d] and top in [1, min(experts, %d)]", 32 * MOE_MAX_PER_LANE, MOE_MAX_TOP);
@@ -269,7 +284,7 @@ extern "C" int b200p_moe_route_scores(const float* logits, int64_t ldl, int32_t*
     if (e != cudaSuccess) return cuda_fail(e, "cudaFuncSetAttribute(moe_route_sigmoid_kernel)");
   }
   moe_route_sigmoid_kernel<<<(unsigned)((M + warps - 1) / warps), warps * 32, smem, st>>>(logits, ldl, nullptr, ids, wts, M, E, top, 1, 1,
-                                                                                           1.f, 0);
+                                                                                           1.f, 0, softmax);
   B200P_LAUNCH_CHECK("moe_route_sigmoid_kernel");
   moe_plan_kernel<<<1, 1024, 2 * E * sizeof(int32_t), st>>>(ids, seg, slot_of, token_of, M * top, E, top);
   B200P_LAUNCH_CHECK("moe_plan_kernel");

@@ -6,7 +6,7 @@
 //   sink_attn_kernel        one token x the query heads of one key/value head, fp32 throughout, any sizes           (per token)
 //   sink_attn_tile_kernel   16 query rows per warp on mma.sync over 64-key tiles: 64 tokens of a prompt for one head, or the
 //                           heads of a key/value head for one decoded token with the keys split over CTAs              (16-bit caches)
-//   sink_attn_merge_kernel  the decode step's partial sums and the sink                                               (per token, head)
+//   attn_merge_kernel       the decode step's partial sums and the sink                                               (per token, head)
 // The softmax starts from the sink: running maximum = sink, running sum = 1 (the sink's own term), accumulator = 0; every key
 // then joins by the usual online update, so a query that sees few keys is damped exactly as the definition says.
 // Every option is a parameter: no norm (weights NULL), no temperature (coef 0), no bias (slope_log2 0), no sink (NULL).
@@ -15,6 +15,7 @@
 // heads' outputs with a sigmoid:
 //   window_attn_prep_kernel  a short causal convolution over time on the q and k projections (carried inputs like the delta
 //                            rule's), q scaled into fp32, k into the cache                                          (per token)
+#include "attn_merge.cuh"
 #include "common.cuh"
 #include "mma_util.cuh"
 
@@ -227,12 +228,11 @@ __global__ void window_attn_prep_kernel(const float* __restrict__ proj, int64_t 
 // run on mma.sync m16n8k16 with the fp32 online softmax in registers, in base-2 units: the distance bias is added to the
 // scores as -slope log2(e) (p - j), and the running maximum / sum start from the sink (max = sink log2(e), sum = 1).
 constexpr int ST_WARPS = 4, ST_THREADS = ST_WARPS * 32, ST_QT = 16 * ST_WARPS, ST_KT = 64, ST_STAGES = 2;
-constexpr float LOG2E = 1.4426950408889634f;
 
 // DECODE = false: 4 warps, rows = 64 consecutive tokens of entry blockIdx.z for head blockIdx.y (tile blockIdx.x of the entry).
 // DECODE = true: ONE warp per CTA; its 16 rows are the query heads of key/value head blockIdx.y for the single token of entry
 // blockIdx.z, and the CTA takes the blockIdx.x-th share of the key tiles (gridDim.x shares): it writes unnormalised partial
-// sums (o, running max, sum; no sink) that sink_attn_merge_kernel combines.  The keys are then read once for all heads of a
+// sums (o, running max, sum; no sink) that attn_merge_kernel (attn_merge.cuh) combines.  The keys are then read once for all heads of a
 // group, by many small CTAs at a time.
 // RULED = true: the scores also pass the ScoreRule (cap, logarithmic penalty, window: tiles before the window of the CTA's first
 // row are skipped, a row whose window has not begun keeps max = -inf and adds nothing) and the output its gate.
@@ -464,34 +464,6 @@ sink_attn_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc, con
   }
 }
 
-// out[e's token, h, :] = out_scale * (sum_s o_s 2^(m_s - m)) / (2^(sink log2e - m) + sum_s l_s 2^(m_s - m)), m the largest of them
-template <typename T>
-__global__ void sink_attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ms,
-                                       const int32_t* __restrict__ cu, const float* __restrict__ sink, T* __restrict__ out,
-                                       int64_t ld_out, float out_scale, int H, int dv, int splits, const float* __restrict__ gate,
-                                       int64_t ldg) {
-  const int e = blockIdx.x, h = blockIdx.y;
-  if (cu[e + 1] - cu[e] <= 0) return;
-  const int64_t base = ((int64_t)e * H + h) * splits;
-  float m = sink ? sink[h] * LOG2E : -INFINITY;
-  for (int sidx = 0; sidx < splits; ++sidx) m = fmaxf(m, part_ms[(base + sidx) * 2]);
-  float den = sink ? exp2f(sink[h] * LOG2E - m) : 0.f;
-  for (int sidx = 0; sidx < splits; ++sidx) {
-    const float ms = part_ms[(base + sidx) * 2];
-    if (ms != -INFINITY) den += part_ms[(base + sidx) * 2 + 1] * exp2f(ms - m);
-  }
-  const float inv = out_scale / den;
-  for (int c = threadIdx.x; c < dv; c += blockDim.x) {
-    float a = 0.f;
-    for (int sidx = 0; sidx < splits; ++sidx) {
-      const float ms = part_ms[(base + sidx) * 2];
-      if (ms != -INFINITY) a = fmaf(part_o[(base + sidx) * dv + c], exp2f(ms - m), a);
-    }
-    const float gz = gate ? sigmoid_f(gate[(int64_t)cu[e] * ldg + (int64_t)h * dv + c]) : 1.f;
-    out[(int64_t)cu[e] * ld_out + (int64_t)h * dv + c] = Tr<T>::from_f(a * inv * gz);
-  }
-}
-
 constexpr int SINK_ATTN_MAX_SPLITS = 16;
 constexpr int SINK_ATTN_MAX_TABLE = 16384;      // longest window whose penalties sit in shared memory (64 KB)
 
@@ -525,9 +497,9 @@ static int sink_attn_tiles_launch(const float* q, const void* kc, const void* vc
     kern<<<grid, 32, smem, st>>>(q, (const T*)kc, (const T*)vc, Tcap, cu, rows, t_pos, sink, slope_log2, (T*)out, ld_out, out_scale,
                                  H, G, part_o, part_ms, rule);
     B200P_LAUNCH_CHECK("sink_attn_tile_kernel");
-    sink_attn_merge_kernel<T><<<dim3((unsigned)nb, (unsigned)H), DV >= 128 ? 128 : 64, 0, st>>>(part_o, part_ms, cu, sink, (T*)out, ld_out,
+    attn_merge_kernel<T><<<dim3((unsigned)nb, (unsigned)H), DV >= 128 ? 128 : 64, 0, st>>>(part_o, part_ms, cu, sink, (T*)out, ld_out,
                                                                                                    out_scale, H, DV, splits, rule.gate, rule.ldg);
-    B200P_LAUNCH_CHECK("sink_attn_merge_kernel");
+    B200P_LAUNCH_CHECK("attn_merge_kernel");
     return B200P_OK;
   }
   auto kern = sink_attn_tile_kernel<T, DK, DV, false, RULED>;

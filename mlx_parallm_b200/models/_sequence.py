@@ -20,11 +20,15 @@ layers mix a recurrent state with windowed attention over a shared low-rank late
     GatedFF                 W_down (act(W_gate x) * W_up x), act in the epilogue     b200p_gemm (fused epilogue)
     ActivatedFF             W_down act(W_up x), act in the epilogue                  b200p_gemm (fused epilogue)
     RoutedExperts           top-k routed GatedFF experts + a shared one; softmax     b200p_moe_* / b200p_gemm_grouped
-                            over the chosen logits, or sigmoid scores picked inside
-                            the best expert groups with a gated shared expert
+                            over the chosen logits, sigmoid scores picked inside
+                            the best expert groups with a gated shared expert, or
+                            plain sigmoid / softmax scores as they are
     LatentAttention         queries and keys/values through low-rank latents,       b200p_latent_prep / b200p_latent_attn
                             sliding window, optional sharing of another layer's latents,  b200p_latent_rope_prep / _q_rope
                             optionally a rotated key part shared by the heads
+    HeadMixAttention        grouped-head attention whose heads' scores are mixed      b200p_mix_attn_prep / b200p_mix_attn
+                            by a matrix before the softmax: biases, q and k normed
+                            as whole rows, partial rotation, sliding window, sink
     WindowAttention         grouped-head attention without rotation over a sliding    b200p_window_attn_prep / b200p_window_attn
                             window: short convolutions on q and k, values that are the
                             keys, capped scores, logarithmic distance penalty, output gate
@@ -35,7 +39,9 @@ layers mix a recurrent state with windowed attention over a shared low-rank late
                             two, with an optional span of layers that runs several times on the same weights
                             (b200p_residual_add_norm), or several copies of the stream that every sublayer reads as a weighted sum
                             and writes back through a mixing matrix, with a tanh norm and a short convolution on what a sublayer
-                            reads (b200p_hyper_step / b200p_canon_conv)
+                            reads (b200p_hyper_step / b200p_canon_conv), or sublayers that read the stream itself and are normed on
+                            their output only, with an optional weighted sum over all layers' results after every layer
+                            (b200p_post_norm_step)
 
 A step is a ragged batch: entry e brings ``counts[e]`` tokens for cache row ``rows[e]``; prompts of different lengths are
 packed back to back (no padding), decode steps bring one token per live row.  Every kernel works from the per-token plan
@@ -46,7 +52,7 @@ softmax, the recurrence and what feeds it are fp32.  A float32 model runs true f
 from __future__ import annotations
 
 import threading
-from typing import Dict, List, Optional, Sequence
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
@@ -54,7 +60,7 @@ from .. import ops
 import math
 
 from .._lib import (GATE_SIGMOID, GATE_SILU, GEMM_GLU_CLAMP, GEMM_GLU_GELU_TANH, GEMM_GLU_SILU, GEMM_RELU_SQ, GEMM_STORE, GEMM_STORE_F32,
-                    SCAN_ACCUMULATE, SCAN_DELTA, SCAN_DELTA_CHANNEL)
+                    GEMM_XIELU, SCAN_ACCUMULATE, SCAN_DELTA, SCAN_DELTA_CHANNEL)
 from .base import BatchedKVCache, ConvTailState, DeltaRuleState, LatentKVCache, RowState, StateGroup, TokenState
 
 MAX_TOKENS_PER_FORWARD = 8192     # packed tokens of one pass through the layers
@@ -67,8 +73,8 @@ class Linear:
         self.in_features, self.out_features = in_features, out_features
         self.weight: Optional[torch.Tensor] = None
 
-    def __call__(self, x, epilogue=GEMM_STORE, out=None, limit=0.0):
-        return ops.gemm(x, self.weight, epilogue, out=out, limit=limit)
+    def __call__(self, x, epilogue=GEMM_STORE, out=None, act=(0.0, 0.0)):
+        return ops.gemm(x, self.weight, epilogue, out=out, act=act)
 
 
 class Scratch:
@@ -406,6 +412,29 @@ def rotary_rates(dims: int, base: float, scaling: Optional[dict] = None) -> List
     return out
 
 
+def stretched_rates(dims: int, base: float, scaling: Optional[dict] = None) -> Tuple[List[float], float]:
+    """(angle per position of pair i, i < dims / 2; factor on cos and sin).  f_i = base^(-2i / dims).  With
+    ``scaling`` (factor, original, fast, slow): d(t) = dims ln(original / (2 pi t)) / (2 ln base) is the (fractional) pair that
+    makes t turns in ``original`` positions; lo = max(floor(d(fast)), 0), hi = min(ceil(d(slow)), dims - 1); pairs below lo keep
+    f_i, pairs above hi get f_i / factor, and between them r_i = (i - lo) / max(hi - lo, 0.001) blends the two linearly.  The
+    magnitude is 0.1 ln(factor) + 1."""
+    rates = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)]
+    if not scaling:
+        return rates, 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+
+    def pair_of(turns: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+
+    lo = max(math.floor(pair_of(float(scaling["fast"]))), 0)
+    hi = min(math.ceil(pair_of(float(scaling["slow"]))), dims - 1)
+    out = []
+    for i, f in enumerate(rates):
+        r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        out.append(f / factor * r + f * (1.0 - r))
+    return out, 0.1 * math.log(factor) + 1.0
+
+
 class DifferentialAttention:
     """Causal attention with ``heads`` query heads over ``kv_heads`` key/value heads and ``maps`` (1 or 2) score maps per head:
     q holds heads x maps vectors of ``dim``, k kv_heads x maps, v kv_heads vectors of ``vdim``; every map is a softmax attention
@@ -592,6 +621,56 @@ class WindowAttention:
         return self.o_proj(mix, GEMM_STORE_F32, out=y_out)
 
 
+class HeadMixAttention:
+    """Causal attention with ``heads`` query heads over ``kv_heads`` key/value heads (query head h reads h // (heads // kv_heads)),
+    keys of ``dim`` and values of ``vdim``, whose heads' scores are mixed before the softmax:
+    score_h = sum_g talk[h, g] (q_g . k_g * scale).  q, k, v carry biases (``bias``); q and k are rms-normed over ALL their heads at
+    once (``row_norm``); the first 2 len(rates) dimensions of every head are rotated by position * rates[i], cos and sin times
+    ``mag``, dimension i paired with i + len(rates) (``pairs``: 2i with 2i + 1); ``window`` > 0: position i sees j with
+    0 <= i - j < window; the softmax denominator also holds exp(sink_h) (``sink`` False: not).  Projection columns [q | k | v]; the
+    rotated keys and the values are cached per position."""
+
+    DECODE_WS_ROWS = 256
+
+    def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, rates: Sequence[float] = (),
+                 mag: float = 1.0, pairs: bool = False, window: int = 0, bias: bool = True, row_norm: bool = True, sink: bool = True):
+        if heads % kv_heads or 2 * len(rates) > dim:
+            raise ValueError("heads must be a multiple of kv_heads and the rotated dimensions at most dim")
+        self.width, self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.eps = width, heads, kv_heads, dim, vdim, float(scale), eps
+        self.rate_values, self.mag, self.pairs, self.window = [float(r) for r in rates], float(mag), bool(pairs), int(window)
+        self.has_bias, self.row_norm, self.has_sink = bool(bias), bool(row_norm), bool(sink)
+        self.col_k = heads * dim
+        self.col_v = self.col_k + kv_heads * dim
+        self.n_proj = self.col_v + kv_heads * vdim
+        self.n_mix = heads * vdim
+        self.in_proj = Linear(width, self.n_proj)
+        self.o_proj = Linear(self.n_mix, width)
+        self.bias = self.q_norm_w = self.k_norm_w = self.talk = self.sink = self.rates = None      # fp32 on the device
+
+    def new_state(self, batch_size: int) -> RowState:
+        return BatchedKVCache(self.dim, self.kv_heads, batch_size, value_dim=self.vdim)
+
+    def reserve(self, s: Scratch, dt):
+        s.reserve("proj", torch.float32, self.n_proj)
+        s.reserve("aq", torch.float32, self.col_k)
+        s.reserve("mix", dt, self.n_mix)
+        if dt != torch.float32:
+            s.reserve_flat("attn_ws", torch.float32, ops.mix_attn_workspace_floats(min(s.rows, self.DECODE_WS_ROWS), self.heads, self.vdim))
+
+    def __call__(self, x, y_out, st: BatchedKVCache, plan: dict, s: Scratch, caches):
+        M, dt, f32 = x.shape[0], x.dtype, torch.float32
+        proj = self.in_proj(x, GEMM_STORE_F32, out=s.get("proj", f32, M, self.n_proj))
+        q = s.get("aq", f32, M, self.col_k)
+        ops.mix_attn_prep(proj, 0, self.col_k, self.col_v, self.bias, self.q_norm_w, self.k_norm_w, self.eps, self.rates, len(self.rate_values),
+                          self.mag, self.pairs, self.scale, q, st.keys, st.values, plan["t_row"], plan["t_pos"], self.heads, self.kv_heads,
+                          self.dim, self.vdim)
+        mix = s.get("mix", dt, M, self.n_mix)
+        ops.mix_attn(q, st.keys, st.values, plan["t_row"], plan["t_pos"], self.talk, self.sink, mix, self.heads, self.kv_heads, self.dim,
+                     self.vdim, window=self.window, cu=plan["cu"], rows=plan["rows"], nb=plan["nb"], max_n=plan["max_n"],
+                     workspace=s.flat("attn_ws", f32) if dt != f32 else None)
+        return self.o_proj(mix, GEMM_STORE_F32, out=y_out)
+
+
 class GatedFF:
     """Feed-forward y = W_down (act(W_gate x) * W_up x) with the gated unit computed in the GEMM epilogue; gate and up rows are
     interleaved in one matrix so that the epilogue holds both values of a hidden unit.  ``act``: "gelu_tanh", "silu", or
@@ -614,7 +693,7 @@ class GatedFF:
         s.reserve("act", dt, self.ff)
 
     def __call__(self, x, y_out, s: Scratch):
-        act = self.gate_up(x, self.epilogue, out=s.get("act", x.dtype, x.shape[0], self.ff), limit=self.limit)
+        act = self.gate_up(x, self.epilogue, out=s.get("act", x.dtype, x.shape[0], self.ff), act=(self.limit, 0.0))
         return self.down(act, GEMM_STORE_F32, out=y_out)
 
 
@@ -624,21 +703,28 @@ class ClampedGLU(GatedFF):
 
 
 class ActivatedFF:
-    """Ungated feed-forward y = W_down act(W_up x) with the activation in the GEMM epilogue; ``act``: "relu_squared"."""
+    """Ungated feed-forward y = W_down act(W_up x) with the activation in the GEMM epilogue; ``act``: "relu_squared", or "xielu"
+    with two learned numbers (p, q): softplus(p) z^2 + z / 2 for z > 0, (1/2 + softplus(q)) (e^z - 1 - z) + z / 2 for z <= 0."""
 
-    EPILOGUES = {"relu_squared": GEMM_RELU_SQ}
+    EPILOGUES = {"relu_squared": GEMM_RELU_SQ, "xielu": GEMM_XIELU}
 
     def __init__(self, width: int, ff: int, act: str):
         self.width, self.ff = width, ff
         self.epilogue = self.EPILOGUES[act]
+        self.act_constants = (0.0, 0.0)
         self.up = Linear(width, ff)
         self.down = Linear(ff, width)
+
+    def set_xielu(self, act: torch.Tensor):
+        """The epilogue's factors from the two learned numbers (computed once on the host in float64)."""
+        p, q = (float(torch.nn.functional.softplus(v)) for v in act.double().cpu())
+        self.act_constants = (p, 0.5 + q)
 
     def reserve(self, s: Scratch, dt):
         s.reserve("act", dt, self.ff)
 
     def __call__(self, x, y_out, s: Scratch):
-        act = self.up(x, self.epilogue, out=s.get("act", x.dtype, x.shape[0], self.ff))
+        act = self.up(x, self.epilogue, out=s.get("act", x.dtype, x.shape[0], self.ff), act=self.act_constants)
         return self.down(act, GEMM_STORE_F32, out=y_out)
 
 
@@ -649,7 +735,8 @@ class RoutedExperts:
       "sigmoid"  scores s = sigmoid(W_r x); experts are picked by s + correction (a vector per layer) among the experts of the
                  ``groups[1]`` best of ``groups[0]`` equal groups of neighbouring experts (a group's score: the sum of its two
                  largest picking scores); weights s / sum(chosen s) * ``route_scale``.
-      "scores"   the ``top`` largest s = sigmoid(W_r x) chosen, their weights those scores as they are.
+      "scores"   the ``top`` largest s = sigmoid(W_r x) chosen, their weights those scores as they are;
+      "softmax_scores"  the same with s = softmax(W_r x) over all experts.
     ``weight_on`` "input": the weight multiplies what the expert reads, y = sum expert_k(w_k x), instead of its output.
     ``limit``: the clamp of experts with the "clamped" unit.
     ``shared_gate``: the shared expert's output is multiplied by sigmoid(w_sg . x), one number per token (w_sg is stacked under
@@ -660,7 +747,7 @@ class RoutedExperts:
     def __init__(self, width: int, experts: int, top: int, ff: int, act: str, shared_ff: int = 0, shared_act: Optional[str] = None,
                  router_bias: bool = True, scoring: str = "softmax", groups: Sequence[int] = (1, 1), route_scale: float = 1.0,
                  shared_gate: bool = False, weight_on: str = "output", limit: float = 0.0):
-        if scoring not in ("softmax", "sigmoid", "scores"):
+        if scoring not in ("softmax", "sigmoid", "scores", "softmax_scores"):
             raise ValueError(f"unknown expert scoring {scoring!r}")
         if weight_on not in ("output", "input"):
             raise ValueError(f"the routing weight goes on the experts' output or input, not {weight_on!r}")
@@ -706,8 +793,9 @@ class RoutedExperts:
         ids, wts = s.get("moe_ids", i32, M, self.top), s.get("moe_wts", f32, M, self.top)
         slot_of, token_of = s.get("moe_slot", i32, M, self.top), s.get("moe_tok", i32, M, self.top)
         seg = s.flat("moe_seg", i32)
-        if self.scoring == "scores":
-            ops.moe_route_scores(logits, ids, wts, seg, slot_of, token_of, self.top, experts=self.experts)
+        if self.scoring in ("scores", "softmax_scores"):
+            ops.moe_route_scores(logits, ids, wts, seg, slot_of, token_of, self.top, experts=self.experts,
+                                 softmax=self.scoring == "softmax_scores")
         elif self.scoring == "sigmoid":
             ops.moe_route_sigmoid(logits, self.router_bias, ids, wts, seg, slot_of, token_of, self.top, self.groups[0], self.groups[1],
                                   self.route_scale, experts=self.experts)
@@ -719,7 +807,7 @@ class RoutedExperts:
             ops.moe_scatter_scaled(x, slot_of, wts, xs, self.top)
         else:
             ops.moe_gather(x, token_of, xs)
-        act = ops.gemm_grouped(xs, self.gate_up, seg, M, self.epilogue, out=s.get("moe_act", dt, n, self.ff), limit=self.limit)
+        act = ops.gemm_grouped(xs, self.gate_up, seg, M, self.epilogue, out=s.get("moe_act", dt, n, self.ff), act=(self.limit, 0.0))
         ye = ops.gemm_grouped(act, self.down, seg, M, GEMM_STORE_F32, out=s.get("moe_y", f32, n, self.width))
         ysh = None
         if self.shared is not None:
@@ -769,11 +857,13 @@ class Sublayer:
 
 
 class LayerRun:
-    """One execution of a layer of the "parallel" or the "prenorm" chain.  "parallel": x <- x + mixer(n(x)) + mlp(n(x)) with ONE
+    """One execution of a layer of the "parallel", the "prenorm" or the "postnorm" chain.  "parallel": x <- x + mixer(n(x)) + mlp(n(x)) with ONE
     norm n (weight ``norm_w``, fp32, applied as a plain factor).  "prenorm": x <- x + mixer(n(x)), then x <- x + mlp(n2(x)) with a
     second norm (``norm2_w``).  ``slot`` is the run's entry in the cache list: a layer that runs several times (a looped span)
     has one run and one state per pass on the same modules.  ``opens``: the run is the first of a pass of the span, which
-    begins with x <- W_in [x ; embedding] (``SequenceModel.loop_in``; models without it leave every ``opens`` False)."""
+    begins with x <- W_in [x ; embedding] (``SequenceModel.loop_in``; models without it leave every ``opens`` False).
+    "postnorm": x <- x + n(mixer(x)), then x <- x + n2(mlp(x)); with ``avg_w`` (fp32 on the device, one number per vector) what goes
+    on is sum_j avg_w[j] X_j over the embedding output X_0 and the results of all runs so far, this one's last."""
 
     def __init__(self, layer: int, slot: int, mixer, mlp, norm_w_name: str, opens: bool = False, norm2_w_name: Optional[str] = None):
         self.layer, self.slot, self.mixer, self.mlp, self.norm_w_name, self.opens = layer, slot, mixer, mlp, norm_w_name, opens
@@ -782,6 +872,7 @@ class LayerRun:
         self.port2: Optional[StreamPort] = None
         self.norm_w: Optional[torch.Tensor] = None
         self.norm2_w: Optional[torch.Tensor] = None
+        self.avg_w: Optional[torch.Tensor] = None
 
 
 class StreamPort:
@@ -813,7 +904,9 @@ class SequenceModel:
     sublayer between two norms; "parallel": ``self.runs`` (LayerRun, in execution order) and optionally ``self.loop_in``;
     "prenorm": ``self.runs`` whose mixer and feed-forward each read a norm of their own; "hyper": ``self.runs`` with a
     ``StreamPort`` per sublayer over ``self.streams`` copies of the stream, a tanh norm (also the model's last one,
-    ``self.final_tanh_norm`` = (alpha, w, b)) and a convolution of ``self.canon_taps`` taps on every sublayer's input.
+    ``self.final_tanh_norm`` = (alpha, w, b)) and a convolution of ``self.canon_taps`` taps on every sublayer's input;
+    "postnorm": ``self.runs`` whose norms stand on the sublayers' outputs, with ``self.embed_norm_w`` (a norm on the embedding) and
+    per-run averages over depth as options.
     ``self.logit_scale`` multiplies the logits."""
 
     block_style = "sandwich"
@@ -841,6 +934,8 @@ class SequenceModel:
         self.eps = 1e-6
         self.logit_scale = 1.0
         self.streams, self.canon_taps = 1, 1          # "hyper" chain
+        self.embed_norm_w: Optional[torch.Tensor] = None      # "postnorm" chain: norm of the embedding (None: not normed)
+        self.depth_average = False                    # "postnorm" chain: the runs have ``avg_w``
         self.final_tanh_norm: Optional[tuple] = None  # (alpha, w, b): the last norm is tanh(alpha x) w + b instead of an rms norm
         # debugging aid: callable(layer, kind, h [M, width]) run after every closed branch of an eager pass (never set it
         # while a decode step is being captured)
@@ -878,7 +973,7 @@ class SequenceModel:
             W, taps = self.args.width, self.canon_taps
             return [StateGroup([r.mixer.new_state(batch_size), ConvTailState(W, taps, batch_size), ConvTailState(W, taps, batch_size)],
                                batch_size) for r in self.runs] + [TokenState(batch_size)]
-        if self.block_style in ("parallel", "prenorm"):
+        if self.block_style in ("parallel", "prenorm", "postnorm"):
             return [r.mixer.new_state(batch_size) for r in self.runs] + [TokenState(batch_size)]
         return [m.new_state(batch_size) for m in self.mixers] + [TokenState(batch_size)]
 
@@ -913,6 +1008,8 @@ class SequenceModel:
             if self.block_style == "hyper":
                 s.reserve("xs", torch.float32, self.streams * W)
                 s.reserve("n", torch.float32, W)
+            if self.depth_average:
+                s.reserve("depth", torch.float32, len(self.runs) * W)
             s.reserve("y", torch.float32, W)
             s.reserve("x", dt, W)
             s.reserve("xl", dt, W)
@@ -954,6 +1051,8 @@ class SequenceModel:
             return self._chain_prenorm(h, x, y, plan, s, cache)
         if self.block_style == "hyper":
             return self._chain_hyper(h, x, y, plan, s, cache, M)
+        if self.block_style == "postnorm":
+            return self._chain_postnorm(h, x, y, plan, s, cache, M)
         subs = self.sublayers
 
         def feed(nxt: Optional[Sublayer], y_in, post_w):
@@ -1066,6 +1165,32 @@ class SequenceModel:
             tap = closes_run and self.residual_tap is not None
             step(y, port, k + 1, k + 1 == len(stops) or tap)
             if tap:
+                self.residual_tap(r.layer, "run", h)
+
+    def _chain_postnorm(self, h, x, y, plan: dict, s: Scratch, cache: List[RowState], M: int):
+        """The runs of a "postnorm" model over the residual stream h (fp32): h += n(mixer(h)), h += n2(mlp(h)), then (with depth
+        averages) h = the weighted sum of the embedding output and all results so far.  Closing a sublayer, keeping a run's result,
+        averaging and writing the storage-type copy that the next sublayer multiplies are ONE pass over the row."""
+        dt, W, eps, runs = self.dtype, self.args.width, self.eps, self.runs
+        # X_0 (the embedding output) .. X_(n-1); the last run's result is only averaged, never read again
+        stack = s.get("depth", torch.float32, M, len(runs) * W).view(M, len(runs), W) if self.depth_average else None
+        if self.embed_norm_w is not None:
+            ops.post_norm_step(h, self.embed_norm_w, eps, dt, stack=stack, slot=0 if stack is not None else -1, raw_out=x)
+        else:
+            ops.norm_add_norm(h, eps, dt, raw_out=x)
+            if stack is not None:
+                stack[:, 0].copy_(h)
+        for i, r in enumerate(runs):
+            last = i + 1 == len(runs)
+            closing = dict(raw_out=None if last else x)
+            if stack is not None:
+                closing.update(stack=stack, slot=-1 if last else i + 1, avg=r.avg_w)
+            r.mixer(x, y, cache[r.slot], plan, s, cache)
+            if r.mlp is not None:
+                ops.post_norm_step(h, r.norm_w, eps, dt, y=y, raw_out=x)
+                r.mlp(x, y, s)
+            ops.post_norm_step(h, r.norm_w if r.mlp is None else r.norm2_w, eps, dt, y=y, **closing)
+            if self.residual_tap is not None:
                 self.residual_tap(r.layer, "run", h)
 
     def _advance_device(self, cache: List[RowState], a: dict, B: int, ids_i32: Optional[torch.Tensor] = None):

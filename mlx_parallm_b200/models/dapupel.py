@@ -25,42 +25,18 @@ The reference has no such graph; the blocks are in models/_sequence.py and run o
 """
 from __future__ import annotations
 
-import math
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional, Tuple
+from typing import Any, Dict, List
 
 import torch
 
 from ._sequence import (GatedDeltaMixer, GatedFF, HashedBigramEmbedding, LatentAttention, LayerRun, Linear, RoutedExperts, SequenceModel,
-                        StreamPort, WindowAttention)
+                        StreamPort, WindowAttention, stretched_rates)
 from .base import BaseModelArgs
 
 MIXER_TYPES = ("channel_delta", "latent_attention", "attention")
 MAX_STREAMS = 8
 MAX_CANON_TAPS = 16
-
-
-def stretched_rates(dims: int, base: float, scaling: Optional[dict] = None) -> Tuple[List[float], float]:
-    """(angle per position of the pairs (2i, 2i+1), i < dims / 2; factor on cos and sin).  f_i = base^(-2i / dims).  With
-    ``scaling`` (factor, original, fast, slow): d(t) = dims ln(original / (2 pi t)) / (2 ln base) is the (fractional) pair that
-    makes t turns in ``original`` positions; lo = max(floor(d(fast)), 0), hi = min(ceil(d(slow)), dims - 1); pairs below lo keep
-    f_i, pairs above hi get f_i / factor, and between them r_i = (i - lo) / max(hi - lo, 0.001) blends the two linearly.  The
-    magnitude is 0.1 ln(factor) + 1."""
-    rates = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)]
-    if not scaling:
-        return rates, 1.0
-    factor, original = float(scaling["factor"]), float(scaling["original"])
-
-    def pair_of(turns: float) -> float:
-        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
-
-    lo = max(math.floor(pair_of(float(scaling["fast"]))), 0)
-    hi = min(math.ceil(pair_of(float(scaling["slow"]))), dims - 1)
-    out = []
-    for i, f in enumerate(rates):
-        r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
-        out.append(f / factor * r + f * (1.0 - r))
-    return out, 0.1 * math.log(factor) + 1.0
 
 
 @dataclass

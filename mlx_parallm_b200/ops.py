@@ -251,10 +251,11 @@ def sample_top_p(logits, temperature, top_p, seed, offset, out=None, probs_out=N
 
 
 # ---- dense linear layers, ragged batches, gated delta rule, latent attention ------------------------------------------
-def gemm(x, w, epilogue=_lib.GEMM_STORE, out=None, limit=0.0, batch=1, strides=(0, 0, 0), M=None, N=None, K=None,
+def gemm(x, w, epilogue=_lib.GEMM_STORE, out=None, act=(0.0, 0.0), batch=1, strides=(0, 0, 0), M=None, N=None, K=None,
          ldx=None, ldw=None, ldy=None):
     """y = x . w^T with fp32 accumulation (b200p_gemm).  Plain call: x [M, K], w [N, K] of one dtype.  Batched call (one
-    weight block per head): pass M, N, K, the row strides and ``strides`` = element strides of x, w, y between products."""
+    weight block per head): pass M, N, K, the row strides and ``strides`` = element strides of x, w, y between products.
+    ``act``: the epilogue's constants (the clamp of GEMM_GLU_CLAMP, the two factors of GEMM_XIELU)."""
     _dev(x, w, out)
     assert x.dtype == w.dtype and x.stride(-1) == 1 and w.stride(-1) == 1
     if M is None:
@@ -270,7 +271,7 @@ def gemm(x, w, epilogue=_lib.GEMM_STORE, out=None, limit=0.0, batch=1, strides=(
     want = torch.float32 if epilogue == _lib.GEMM_STORE_F32 else x.dtype
     assert out.dtype == want and out.stride(-1) == 1, (out.dtype, want)
     _call(("b200p_gemm", N, K, batch), lambda: lib().b200p_gemm(_p(x), _p(w), _p(out), M, N, K, ldx, ldw, ldy, batch, strides[0], strides[1],
-                                                        strides[2], dtype_code(x.dtype), epilogue, float(limit), _stream()))
+                                                        strides[2], dtype_code(x.dtype), epilogue, float(act[0]), float(act[1]), _stream()))
     return out
 
 
@@ -364,7 +365,7 @@ def linear_attn_prep(proj, head_decay, q, k, v, decay, H, dk, dv):
                                                                         _p(decay), M, H, dk, dv, _stream()))
 
 
-def gemm_grouped(x, w, seg, max_rows: int, epilogue=_lib.GEMM_STORE, out=None, limit=0.0):
+def gemm_grouped(x, w, seg, max_rows: int, epilogue=_lib.GEMM_STORE, out=None, act=(0.0, 0.0)):
     """Rows [seg[z], seg[z+1]) of x times the z-th block of w [groups, N, K] (b200p_gemm_grouped); ``seg`` int32 on the device."""
     _dev(x, w, seg, out)
     groups, N, K = w.shape
@@ -376,8 +377,7 @@ def gemm_grouped(x, w, seg, max_rows: int, epilogue=_lib.GEMM_STORE, out=None, l
     assert out.dtype == want and out.stride(-1) == 1
     _call(("b200p_gemm_grouped", N, K, groups), lambda: lib().b200p_gemm_grouped(
         _p(x), _p(w), _p(out), _p(seg), x.shape[0], int(max_rows), N, K, x.stride(0), K, out.stride(0), groups, N * K, dtype_code(x.dtype),
-        epilogue,
-        float(limit), _stream()))
+        epilogue, float(act[0]), float(act[1]), _stream()))
     return out
 
 
@@ -617,14 +617,14 @@ def window_attn(q, kcache, vcache, t_row, t_pos, out, H, G, dk, dv, softcap=0.0,
     return out
 
 
-def moe_route_scores(logits, ids, wts, seg, slot_of, token_of, top: int, experts: Optional[int] = None):
-    """Routing by the largest sigmoid scores; the weights are the scores themselves."""
+def moe_route_scores(logits, ids, wts, seg, slot_of, token_of, top: int, experts: Optional[int] = None, softmax: bool = False):
+    """Routing by the largest sigmoid scores, or the largest of a softmax over all experts; the weights are the scores themselves."""
     _dev(logits, ids, wts, seg, slot_of, token_of)
     M = logits.shape[0]
     E = logits.shape[1] if experts is None else int(experts)
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     _call("b200p_moe_route_scores", lambda: lib().b200p_moe_route_scores(_p(logits), logits.stride(0), _p(ids), _p(wts), _p(seg), _p(slot_of),
-                                                                        _p(token_of), M, E, int(top), _stream()))
+                                                                        _p(token_of), M, E, int(top), int(softmax), _stream()))
 
 
 def moe_scatter_scaled(x, slot_of, wts, xs, top: int):
@@ -673,3 +673,51 @@ def tanh_norm(h, alpha, w, b, x_out):
     assert h.dtype == torch.float32 and h.is_contiguous() and x_out.is_contiguous()
     _call("b200p_tanh_norm", lambda: lib().b200p_tanh_norm(_p(h), _p(alpha), _p(w), _p(b), _p(x_out), M, W, dtype_code(x_out.dtype),
                                                           _stream()))
+
+
+def post_norm_step(h, w, eps, dtype, y=None, stack=None, slot=-1, avg=None, raw_out=None):
+    """Close a sublayer that is normed on its output: x = h + rms_norm(y) * w (``y`` None: x = rms_norm(h) * w), kept in
+    ``stack`` [M, slots, W] at ``slot``; h = x, or with ``avg`` (fp32 [n] on the device) h = sum_j avg[j] stack[:, j] over the first
+    n - 1 slots + avg[n - 1] x; raw_out = h in ``dtype``."""
+    _dev(h, w, y, stack, avg, raw_out)
+    M, W = h.shape
+    for t in (h, w, y, stack, avg):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
+    assert raw_out is None or (raw_out.dtype == dtype and raw_out.is_contiguous())
+    assert stack is None or (stack.dim() == 3 and stack.shape[0] == M and stack.shape[2] == W)
+    _call("b200p_post_norm_step", lambda: lib().b200p_post_norm_step(
+        _p(y), _p(w), _p(h), _p(stack), 0 if stack is None else stack.shape[1], int(slot), _p(avg), 0 if avg is None else avg.numel(),
+        _p(raw_out), M, W, float(eps), dtype_code(dtype), _stream()))
+
+
+def mix_attn_prep(proj, col_q, col_k, col_v, bias, wq, wk, eps, rates, n_rot, mag, pairs, scale, q_out, kcache, vcache, t_row, t_pos, H, G,
+                  dk, dv):
+    """Biased, normed (whole rows), rotated, scaled queries to ``q_out`` fp32 [M, H dk]; keys and values into the caches
+    [rows, G, Tcap, dk] / [rows, G, Tcap, dv] at every token's (row, position)."""
+    _dev(proj, bias, wq, wk, rates, q_out, kcache, vcache, t_row, t_pos)
+    M = proj.shape[0]
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and kcache.is_contiguous() and vcache.is_contiguous() and q_out.is_contiguous()
+    assert kcache.dtype == vcache.dtype and kcache.shape[1:] == (G, kcache.shape[2], dk) and vcache.shape[1:] == (G, kcache.shape[2], dv)
+    assert (wq is None or wq.numel() == H * dk) and (wk is None or wk.numel() == G * dk) and (n_rot == 0 or rates.numel() == n_rot)
+    _call("b200p_mix_attn_prep", lambda: lib().b200p_mix_attn_prep(
+        _p(proj), proj.stride(0), int(col_q), int(col_k), int(col_v), _p(bias), _p(wq), _p(wk), float(eps), _p(rates), int(n_rot), float(mag),
+        int(pairs), float(scale), _p(q_out), _p(kcache), _p(vcache), kcache.shape[2], _p(t_row), _p(t_pos), M, H, G, dk, dv,
+        dtype_code(kcache.dtype), _stream()))
+
+
+def mix_attn_workspace_floats(nb: int, H: int, dv: int) -> int:
+    return lib().b200p_mix_attn_workspace_bytes(nb, H, dv) // 4
+
+
+def mix_attn(q, kcache, vcache, t_row, t_pos, talk, sink, out, H, G, dk, dv, window=0, cu=None, rows=None, nb=0, max_n=1, workspace=None):
+    """Attention whose heads' scores are mixed by ``talk`` fp32 [H, H] before the softmax, with a window and a sink (both
+    optional); ``out`` [M, >= H * dv] in the caches' dtype.  ``workspace`` (fp32): partial sums of a decode step."""
+    _dev(q, kcache, vcache, t_row, t_pos, talk, sink, out, cu, rows, workspace)
+    M = q.shape[0]
+    assert q.dtype == torch.float32 and q.is_contiguous() and out.stride(1) == 1 and out.dtype == kcache.dtype
+    assert talk.dtype == torch.float32 and talk.is_contiguous() and talk.shape == (H, H)
+    _call("b200p_mix_attn", lambda: lib().b200p_mix_attn(
+        _p(q), _p(kcache), _p(vcache), kcache.shape[2], _p(t_row), _p(t_pos), _p(cu), _p(rows), int(nb), int(max_n), _p(talk), _p(sink),
+        int(window), _p(out), out.stride(0), M, H, G, dk, dv, dtype_code(kcache.dtype), _p(workspace),
+        0 if workspace is None else workspace.numel() * 4, _stream()))
+    return out

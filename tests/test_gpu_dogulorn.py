@@ -88,7 +88,7 @@ def test_gemm_gated_epilogue_and_heads(dtype, M):
     a = torch.clamp(x.double() @ gate.double().T, max=lim)
     u = torch.clamp(x.double() @ up.double().T, -lim, lim)
     want = a * torch.sigmoid(1.702 * a) * (u + 1)
-    got = ops.gemm(x.cuda(), gu.cuda().contiguous(), _lib.GEMM_GLU_CLAMP, limit=lim)
+    got = ops.gemm(x.cuda(), gu.cuda().contiguous(), _lib.GEMM_GLU_CLAMP, act=(lim, 0.0))
     assert got.shape == (M, F) and (got.double().cpu() - want).abs().max() < (1e-4 if dtype == torch.float32 else 0.04)
     # one weight block per head, operands strided inside wider rows
     H, dk, R = 3, 8, 16
@@ -129,7 +129,7 @@ def test_gemm_tcgen05_tiles(dtype, M, N, K):
         lim = 0.7
         a = torch.clamp(want[:, 0::2], max=lim)
         u = torch.clamp(want[:, 1::2], -lim, lim)
-        glu = ops.gemm(x, w, _lib.GEMM_GLU_CLAMP, limit=lim)
+        glu = ops.gemm(x, w, _lib.GEMM_GLU_CLAMP, act=(lim, 0.0))
         assert glu.shape == (M, N // 2) and (glu.double() - a * torch.sigmoid(1.702 * a) * (u + 1)).abs().max() < 0.02
 
 
