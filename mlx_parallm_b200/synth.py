@@ -626,3 +626,86 @@ def dapupel_random_weights(cfg: dict, seed: int = 1234, device="cpu", rank: Opti
             t = 1.0 + 0.02 * torch.randn(shape, generator=g, device=dev)
         out[name] = t.to(torch.bfloat16)
     return out
+
+
+# ---- Seradra ----------------------------------------------------------------------------------------------------------------
+def seradra_config(width: int, ff: int, n_layers: int, heads: int, head_dim: int, q_rank: int, kv_rank: int, window: int,
+                   kv_heads: Optional[int] = None, rot_dim: int = 64, experts: int = 16, top: int = 2, vocab: int = 32000, **unused) -> dict:
+    """A config of the design at the sizes of a real model: layers cycle (mixed-score attention with a dense feed-forward,
+    latent attention with routed experts, mixed-score attention with routed experts); the experts a token uses together have the
+    hidden size ``ff``; half of every head is rotated."""
+    kv_heads = kv_heads or max(1, heads // 4)
+    scaling = {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5, "mask": {"size": window},
+                 "rot": {"dims": head_dim // 2, "base": 500000.0, "scaling": scaling}}
+    latent = {"heads": heads, "dim": head_dim, "rot_dim": rot_dim, "vdim": head_dim, "q_rank": q_rank, "kv_rank": kv_rank,
+              "scale": (head_dim + rot_dim) ** -0.5, "mask": {"size": window}, "rot": {"dims": rot_dim, "base": 10000.0}}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff // top}}
+    layers = []
+    for i in range(n_layers):
+        layers.append({"type": "latent_attention" if i % 3 == 1 else "attention", "mixer": dict(latent if i % 3 == 1 else attention),
+                       "mlp": {"kind": "dense", "ff": ff} if i % 3 == 0 else moe})
+    return {"architecture": "Seradra", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": 1e-6}}
+
+
+def seradra_shapes(cfg: dict) -> Dict[str, tuple]:
+    """Shape of every tensor of a Seradra checkpoint (matrices [out, in])."""
+    W, V = cfg["width"], cfg["vocab"]
+    out = {"embed": (V, W), "embed.norm": (W,), "final.norm": (W,), "head": (V, W)}
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.mix.", L["mixer"]
+        H = m["heads"]
+        out[f"l{i}.norm1"], out[f"l{i}.dwa"] = (W,), (i + 2,)
+        if L["type"] == "attention":
+            G = m.get("kv_heads", H)
+            for n, rows in (("q", H * m["dim"]), ("k", G * m["dim"]), ("v", G * m["vdim"])):
+                out[p + n], out[f"{p}{n}.b"] = (rows, W), (rows,)
+                if n != "v":
+                    out[f"{p}{n}.norm"] = (rows,)
+            out[p + "talk"], out[p + "sink"], out[p + "o"] = (H, H), (H,), (W, H * m["vdim"])
+        else:
+            out[p + "dq"], out[p + "dq.norm"], out[p + "uq"] = (m["q_rank"], W), (m["q_rank"],), (H * (m["dim"] + m["rot_dim"]), m["q_rank"])
+            out[p + "dkv"], out[p + "dkv.norm"] = (m["kv_rank"] + m["rot_dim"], W), (m["kv_rank"],)
+            out[p + "uk"], out[p + "uv"], out[p + "o"] = (H * m["dim"], m["kv_rank"]), (H * m["vdim"], m["kv_rank"]), (W, H * m["vdim"])
+        mlp = L.get("mlp")
+        if mlp is None:
+            continue
+        q = f"l{i}.mlp."
+        out[f"l{i}.norm2"] = (W,)
+        if mlp["kind"] == "dense":
+            out[q + "up"], out[q + "down"], out[q + "act"] = (mlp["ff"], W), (W, mlp["ff"]), (2,)
+        else:
+            for e in range(mlp["router"]["experts"]):
+                out[f"{q}e{e}.gate"] = out[f"{q}e{e}.up"] = (mlp["expert"]["ff"], W)
+                out[f"{q}e{e}.down"] = (W, mlp["expert"]["ff"])
+            out[q + "router"] = (mlp["router"]["experts"], W)
+    return out
+
+
+def seradra_random_weights(cfg: dict, seed: int = 1234, device="cpu") -> Dict[str, torch.Tensor]:
+    """bfloat16 tensors: matrices N(0, 1/in), score mixing near the identity, norm weights near their neutral value, depth averages
+    near "the last result only", biases, sinks and activation parameters small."""
+    dev = torch.device(device)
+    out: Dict[str, torch.Tensor] = {}
+    for name, shape in seradra_shapes(cfg).items():
+        g = torch.Generator(device=dev)
+        g.manual_seed(_stable_seed(seed, name))
+        leaf = name.split(".")[-1]
+        r = torch.randn(shape, generator=g, device=dev)
+        if leaf == "talk":
+            t = torch.eye(shape[0], device=dev) + r * (0.2 / math.sqrt(shape[0]))
+        elif leaf == "dwa":
+            t = r * 0.05
+            t[-1] += 1.0
+        elif name == "embed":
+            t = r
+        elif len(shape) == 2:
+            t = r / math.sqrt(shape[1])
+        elif leaf in ("b", "sink", "act"):
+            t = r * 0.1
+        elif leaf in ("norm1", "norm2") or name in ("embed.norm", "final.norm"):
+            t = r * 0.02
+        else:                                   # q.norm, k.norm, dq.norm, dkv.norm
+            t = 1.0 + r * 0.02
+        out[name] = t.to(torch.bfloat16)
+    return out
