@@ -16,6 +16,17 @@
 
 namespace b200p {
 
+// V fp32 values into V neighbouring cache elements (V == 4: one 8- or 16-byte store)
+template <typename T, int V>
+__device__ __forceinline__ void store_cache(T* d, const float (&x)[V]) {
+  if constexpr (V == 4 && sizeof(T) == 2) {
+    *reinterpret_cast<uint2*>(d) = make_uint2(pack2<T>(x[0], x[1]), pack2<T>(x[2], x[3]));
+  } else {
+#pragma unroll
+    for (int k = 0; k < V; ++k) d[k] = Tr<T>::from_f(x[k]);
+  }
+}
+
 // V neighbouring channels per access (4: every head starts on a 16-byte boundary and a rotated group of 4 stays inside its half)
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
@@ -23,11 +34,13 @@ mix_attn_prep_kernel(const float* __restrict__ proj, int64_t ldp, int64_t col_q,
                      const float* __restrict__ bias, const float* __restrict__ wq, const float* __restrict__ wk, float eps,
                      const float* __restrict__ rates, int n_rot, float mag, int pairs, float scale, float* __restrict__ q_out,
                      T* __restrict__ kcache, T* __restrict__ vcache, int64_t Tcap, const int32_t* __restrict__ t_row,
-                     const int32_t* __restrict__ t_pos, int H, int G, int dk, int dv) {
-  extern __shared__ float mp_sm[];                                 // cos, sin of this position: [n_rot] each
+                     const int32_t* __restrict__ t_pos, int H, int G, int dk, int dv, int buffered) {
+  // the biased q | k row (buffered: read once from memory, afterwards from here), cos and sin of this position ([n_rot] each)
+  extern __shared__ __align__(16) float mp_sm[];
   __shared__ float red[2][8];
-  float* cs = mp_sm;
-  float* sn = mp_sm + n_rot;
+  float* rowbuf = mp_sm;
+  float* cs = mp_sm + (buffered ? (H + G) * dk : 0);
+  float* sn = cs + n_rot;
   const int64_t t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int64_t pos = t_pos[t], row = t_row[t];
@@ -52,19 +65,27 @@ mix_attn_prep_kernel(const float* __restrict__ proj, int64_t ldp, int64_t col_q,
   };
   const int nq = H * dk, nk = G * dk;
   float sq = 0.f, sk = 0.f;
-  if (wq)
-    for (int c = threadIdx.x * V; c < nq; c += blockDim.x * V) {
-      float r[V];
-      load(col_q + c, r);
+  if (wq || wk || buffered) {
+#pragma unroll 4
+    for (int c = threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
+      float r[V], ss = 0.f;
+      load(c < nq ? col_q + c : col_k + c - nq, r);
+      if (buffered) {
+        if constexpr (V == 4) *reinterpret_cast<float4*>(rowbuf + c) = make_float4(r[0], r[1], r[2], r[3]);
+        else rowbuf[c] = r[0];
+      }
 #pragma unroll
-      for (int k = 0; k < V; ++k) sq = fmaf(r[k], r[k], sq);
+      for (int k = 0; k < V; ++k) ss = fmaf(r[k], r[k], ss);
+      if (c < nq) sq += ss;
+      else sk += ss;
     }
-  if (wk)
-    for (int c = threadIdx.x * V; c < nk; c += blockDim.x * V) {
+  }
+  const bool in_cache = pos < Tcap;                                // the host sizes the cache first; never write outside it
+  if (in_cache)                                                    // the values need no norm: their reads overlap the reduction
+    for (int c = threadIdx.x * V; c < G * dv; c += blockDim.x * V) {
       float r[V];
-      load(col_k + c, r);
-#pragma unroll
-      for (int k = 0; k < V; ++k) sk = fmaf(r[k], r[k], sk);
+      load(col_v + c, r);
+      store_cache<T, V>(vcache + ((row * G + c / dv) * Tcap + pos) * dv + c % dv, r);
     }
   sq = warp_sum(sq);
   sk = warp_sum(sk);
@@ -73,27 +94,38 @@ mix_attn_prep_kernel(const float* __restrict__ proj, int64_t ldp, int64_t col_q,
   sq = sk = 0.f;
   for (int i = 0; i < nw; ++i) { sq += red[0][i]; sk += red[1][i]; }
   const float inv_q = wq ? 1.f / sqrtf(sq / (float)nq + eps) : 1.f, inv_k = wk ? 1.f / sqrtf(sk / (float)nk + eps) : 1.f;
-  const bool in_cache = pos < Tcap;                                // the host sizes the cache first; never write outside it
+  auto take = [&](int c, float (&r)[V]) {                          // entry c of the q | k row
+    if (!buffered) load(c < nq ? col_q + c : col_k + c - nq, r);
+    else if constexpr (V == 4) {
+      const float4 q4 = *reinterpret_cast<const float4*>(rowbuf + c);
+      r[0] = q4.x; r[1] = q4.y; r[2] = q4.z; r[3] = q4.w;
+    } else r[0] = rowbuf[c];
+  };
   for (int c = threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
     const bool is_q = c < nq;
     const int cc = is_q ? c : c - nq;
     const int head = cc / dk, i = cc % dk;
-    const int64_t col = is_q ? col_q : col_k;
     const float* w = is_q ? wq : wk;
     const float inv = is_q ? inv_q : inv_k;
     float x[V];
-    load(col + cc, x);
-#pragma unroll
-    for (int k = 0; k < V; ++k) x[k] *= inv * (w ? w[cc + k] : 1.f);
+    take(c, x);
+    auto normed = [&](int col, float (&r)[V]) {
+      if (!w) return;
+      if constexpr (V == 4) {
+        const float4 w4 = *reinterpret_cast<const float4*>(w + col);
+        r[0] *= inv * w4.x; r[1] *= inv * w4.y; r[2] *= inv * w4.z; r[3] *= inv * w4.w;
+      } else r[0] *= inv * w[col];
+    };
+    normed(cc, x);
     if (i < 2 * n_rot) {                                           // rotated: u' = u cos - v sin, v' = v cos + u sin
       const bool first = pairs ? (i & 1) == 0 : i < n_rot;
       const int f = pairs ? i >> 1 : (first ? i : i - n_rot);
       const int other = pairs ? cc ^ 1 : (first ? cc + n_rot : cc - n_rot);     // heads start at even columns: cc ^ 1 is the partner
       float o[V];
-      load(col + other, o);
+      take(c + other - cc, o);
+      normed(other, o);
 #pragma unroll
       for (int k = 0; k < V; ++k) {
-        o[k] *= inv * (w ? w[other + k] : 1.f);
         x[k] = first ? x[k] * cs[f + k] - o[k] * sn[f + k] : x[k] * cs[f + k] + o[k] * sn[f + k];
       }
     }
@@ -102,16 +134,9 @@ mix_attn_prep_kernel(const float* __restrict__ proj, int64_t ldp, int64_t col_q,
       if constexpr (V == 4) *reinterpret_cast<float4*>(d) = make_float4(x[0] * scale, x[1] * scale, x[2] * scale, x[3] * scale);
       else d[0] = x[0] * scale;
     } else if (in_cache) {
-      T* d = kcache + ((row * G + head) * Tcap + pos) * dk + i;
-#pragma unroll
-      for (int k = 0; k < V; ++k) d[k] = Tr<T>::from_f(x[k]);
+      store_cache<T, V>(kcache + ((row * G + head) * Tcap + pos) * dk + i, x);
     }
   }
-  if (in_cache)
-    for (int c = threadIdx.x; c < G * dv; c += blockDim.x) {
-      const int g = c / dv, i = c % dv;
-      vcache[((row * G + g) * Tcap + pos) * dv + i] = Tr<T>::from_f(pt[col_v + c] + (bias ? bias[col_v + c] : 0.f));
-    }
 }
 
 // ---- one token per CTA -----------------------------------------------------------------------------------------------------
@@ -706,8 +731,9 @@ static int mix_attn_decode_launch(const float* q, const void* kc, const void* vc
   }
   const size_t smem = md_smem(H, G, DK, DV, KT);
   // as many shares as fill the SMs once
-  const int64_t resident = 148 * (int64_t)(smem > 110 * 1024 ? 1 : smem > 72 * 1024 ? 2 : smem > 54 * 1024 ? 3 : 4);
-  int splits = (int)(resident / M);
+  int per_sm = 1;
+  if (cudaOccupancyMaxActiveBlocksPerMultiprocessor(&per_sm, kern, MD_THREADS, smem) != cudaSuccess || per_sm < 1) per_sm = 1;
+  int splits = (int)(148 * (int64_t)per_sm / M);
   splits = splits < 1 ? 1 : splits > MX_MAX_SPLITS ? MX_MAX_SPLITS : splits;
   const size_t per_split = (size_t)M * H * (DV + 2) * sizeof(float);
   if ((size_t)splits * per_split > ws_bytes) splits = (int)(ws_bytes / per_split);
@@ -852,18 +878,21 @@ extern "C" int b200p_mix_attn_prep(const float* proj, int64_t ldp, int64_t col_q
   B200P_REQUIRE(n_rot >= 0 && 2 * n_rot <= dk && n_rot <= 4096 && (n_rot == 0 || rates), B200P_ERR_ARG, "at most dk dimensions are rotated");
   B200P_REQUIRE(!(pairs && n_rot) || dk % 2 == 0, B200P_ERR_ARG, "pairwise rotation needs heads of an even size");
   if (M == 0) return B200P_OK;
-  const bool vec = !pairs && dk % 4 == 0 && n_rot % 4 == 0 && ldp % 4 == 0 && col_q % 4 == 0 && col_k % 4 == 0 && aligned(proj, 16) &&
+  const bool vec = !pairs && dk % 4 == 0 && dv % 4 == 0 && n_rot % 4 == 0 && ldp % 4 == 0 && col_q % 4 == 0 && col_k % 4 == 0 && col_v % 4 == 0 &&
+                   aligned(wq, 16) && aligned(wk, 16) && aligned(kcache, 16) && aligned(vcache, 16) && aligned(proj, 16) &&
                    aligned(bias, 16) && aligned(q_out, 16);
-  const size_t smem = 2 * (size_t)n_rot * sizeof(float);
+  const size_t turns = 2 * (size_t)n_rot * sizeof(float), row_bytes = (size_t)(H + G) * dk * sizeof(float);
+  const int buffered = turns + row_bytes <= 47 * 1024;
+  const size_t smem = turns + (buffered ? row_bytes : 0);
   cudaStream_t st = (cudaStream_t)stream;
   if (vec) {
     B200P_DISPATCH_DTYPE(dtype, T, (mix_attn_prep_kernel<T, 4><<<(unsigned)M, 256, smem, st>>>(
         proj, ldp, col_q, col_k, col_v, bias, wq, wk, eps, rates, n_rot, mag, pairs, scale, q_out, (T*)kcache, (T*)vcache, Tcap, t_row, t_pos,
-        H, G, dk, dv)));
+        H, G, dk, dv, buffered)));
   } else {
     B200P_DISPATCH_DTYPE(dtype, T, (mix_attn_prep_kernel<T, 1><<<(unsigned)M, 256, smem, st>>>(
         proj, ldp, col_q, col_k, col_v, bias, wq, wk, eps, rates, n_rot, mag, pairs, scale, q_out, (T*)kcache, (T*)vcache, Tcap, t_row, t_pos,
-        H, G, dk, dv)));
+        H, G, dk, dv, buffered)));
   }
   B200P_LAUNCH_CHECK("mix_attn_prep_kernel");
   return B200P_OK;

@@ -5,7 +5,8 @@
 //   stack[slot] = x                     (slot >= 0: x is one of the vectors the averages read)
 //   h = sum_{j < n - 1} a_j stack[j] + a_{n-1} x     (a given; otherwise h = x)
 //   raw_out = h in the storage type     (what the next sublayer multiplies)
-// Everything is fp32 except raw_out.  The stack lies token by token, [M, slots, W].
+// Everything is fp32 except raw_out.  The stack lies token by token, [M, slots, W]: `slot` is none of the slots that
+// the average reads.
 #include "common.cuh"
 
 namespace b200p {
@@ -13,14 +14,14 @@ namespace b200p {
 // V neighbouring channels per access (4: 16 bytes), ITEMS accesses per thread; the row stays in registers between the norm's
 // sum of squares and the result
 template <typename T, int V, int ITEMS>
-__global__ void __launch_bounds__(1024)
+__global__ void __launch_bounds__(ITEMS <= 2 ? 1024 : 512)
 post_norm_step_kernel(const float* __restrict__ y, const float* __restrict__ w, float* __restrict__ h, float* __restrict__ stack,
                       int64_t slots, int slot, const float* __restrict__ a, int n, T* __restrict__ raw_out, int64_t W, float eps) {
   __shared__ float red[32];
   const int64_t t = blockIdx.x;
   float* hr = h + t * W;
   const float* src = y ? y + t * W : hr;
-  float x[ITEMS][V], ss = 0.f;
+  float x[ITEMS][V], hv[ITEMS][V], acc[ITEMS][V], ss = 0.f;
   auto load = [&](const float* p, float (&r)[V]) {
     if constexpr (V == 4) {
       const float4 q = *reinterpret_cast<const float4*>(p);
@@ -33,46 +34,49 @@ post_norm_step_kernel(const float* __restrict__ y, const float* __restrict__ w, 
     if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(r[0], r[1], r[2], r[3]);
     else *p = r[0];
   };
+  // everything that does not wait for the norm's sum is read before it: the row, the stream, the weighted vectors of the stack
 #pragma unroll
   for (int i = 0; i < ITEMS; ++i) {
     const int64_t c = ((int64_t)i * blockDim.x + threadIdx.x) * V;
-    if (c < W) {
-      load(src + c, x[i]);
 #pragma unroll
-      for (int k = 0; k < V; ++k) ss = fmaf(x[i][k], x[i][k], ss);
+    for (int k = 0; k < V; ++k) acc[i][k] = hv[i][k] = x[i][k] = 0.f;
+    if (c >= W) continue;
+    load(src + c, x[i]);
+    if (y) load(hr + c, hv[i]);
+    if (a) {
+      const float* st = stack + t * slots * W + c;
+#pragma unroll 4
+      for (int j = 0; j < n - 1; ++j) {
+        float v[V];
+        load(st + (int64_t)j * W, v);
+#pragma unroll
+        for (int k = 0; k < V; ++k) acc[i][k] = fmaf(a[j], v[k], acc[i][k]);
+      }
     }
   }
+#pragma unroll
+  for (int i = 0; i < ITEMS; ++i)
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss = fmaf(x[i][k], x[i][k], ss);
   ss = warp_sum(ss);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   if (lane == 0) red[warp] = ss;
   __syncthreads();
   float total = 0.f;
   for (int i = 0; i < nw; ++i) total += red[i];      // same order in every thread
-  const float inv = 1.f / sqrtf(total / (float)W + eps);
+  const float inv = 1.f / sqrtf(total / (float)W + eps), last = a ? a[n - 1] : 1.f;
 #pragma unroll
   for (int i = 0; i < ITEMS; ++i) {
     const int64_t c = ((int64_t)i * blockDim.x + threadIdx.x) * V;
     if (c >= W) continue;
-    float wv[V], hv[V];
+    float wv[V];
     load(w + c, wv);
-    if (y) load(hr + c, hv);
 #pragma unroll
-    for (int k = 0; k < V; ++k) x[i][k] = y ? hv[k] + x[i][k] * inv * wv[k] : x[i][k] * inv * wv[k];
-    float* st = stack ? stack + t * slots * W + c : nullptr;
-    if (slot >= 0) store(st + (int64_t)slot * W, x[i]);
+    for (int k = 0; k < V; ++k) x[i][k] = hv[i][k] + x[i][k] * inv * wv[k];          // hv is zero without y
+    if (slot >= 0) store(stack + (t * slots + slot) * W + c, x[i]);
     if (a) {
-      float acc[V];
 #pragma unroll
-      for (int k = 0; k < V; ++k) acc[k] = 0.f;
-#pragma unroll 4
-      for (int j = 0; j < n - 1; ++j) {
-        float v[V];
-        load(st + (int64_t)j * W, v);
-#pragma unroll
-        for (int k = 0; k < V; ++k) acc[k] = fmaf(a[j], v[k], acc[k]);
-      }
-#pragma unroll
-      for (int k = 0; k < V; ++k) x[i][k] = fmaf(a[n - 1], x[i][k], acc[k]);
+      for (int k = 0; k < V; ++k) x[i][k] = fmaf(last, x[i][k], acc[i][k]);
     }
     store(hr + c, x[i]);
     if (raw_out) {
@@ -97,7 +101,8 @@ static int post_norm_step_launch(const float* y, const float* w, float* h, float
   // many tokens: CTAs of at most 256 threads with several pieces each; few tokens (a decode step): a row over more threads
   int64_t threads = M >= 512 ? 256 : 1024;
   if (pieces < threads) threads = (pieces + 31) / 32 * 32;
-  while ((pieces + threads - 1) / threads > POST_NORM_MAX_ITEMS && threads < 1024) threads *= 2;
+  while ((pieces + threads - 1) / threads > 4 && threads < 512) threads *= 2;
+  if ((pieces + threads - 1) / threads > 2 && threads > 512) threads = 512;          // what the kernels of 4 and 8 pieces take
   const int64_t items = (pieces + threads - 1) / threads;
   B200P_REQUIRE(items <= POST_NORM_MAX_ITEMS, B200P_ERR_ARG, "rows of %lld values are not built", (long long)W);
 #define PN_CASE(I_)                                                                                                          \
