@@ -73,6 +73,18 @@ __device__ __forceinline__ float gelu_tanh_unit(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 __device__ __forceinline__ bool gemm_epi_is_glu(int epi) { return epi >= B200P_GEMM_GLU_CLAMP && epi <= B200P_GEMM_GLU_SILU; }
+// act.x z^2 + z / 2 above zero, act.y (e^z - 1 - z) + z / 2 at and below it, without a branch (an epilogue thread then interleaves
+// its elements): e^z - 1 - z is the exponential series from z^2 / 2 on down to -1/4 (what is left out is below 1e-7 of the result),
+// the plain difference below
+__device__ __forceinline__ float xielu_unit(float v, float2 act) {
+  const float up = fmaxf(v, 0.f), dn = fminf(v, 0.f);
+  float p = fmaf(dn, 1.f / 720.f, 1.f / 120.f);
+  p = fmaf(dn, p, 1.f / 24.f);
+  p = fmaf(dn, p, 1.f / 6.f);
+  p = fmaf(dn, p, 0.5f);
+  const float g = dn > -0.25f ? dn * dn * p : __expf(dn) - 1.f - dn;
+  return fmaf(act.x * up, up, fmaf(act.y, g, 0.5f * v));
+}
 // value stored by the ungated epilogues that write the storage type: the accumulator itself, or an activation of it
 // (act: the epilogue's constants)
 __device__ __forceinline__ float gemm_store_act(float v, int epi, float2 act) {
@@ -80,8 +92,7 @@ __device__ __forceinline__ float gemm_store_act(float v, int epi, float2 act) {
     v = fmaxf(v, 0.f);
     return v * v;
   }
-  if (epi == B200P_GEMM_XIELU)       // act.x v^2 + v / 2 above zero, act.y (e^v - 1 - v) + v / 2 below: expm1f keeps small |v| exact
-    return v > 0.f ? fmaf(act.x * v, v, 0.5f * v) : fmaf(act.y, expm1f(v) - v, 0.5f * v);
+  if (epi == B200P_GEMM_XIELU) return xielu_unit(v, act);
   return v;
 }
 __device__ __forceinline__ float glu_unit(float gate, float up, int epi, float2 act) {

@@ -99,7 +99,14 @@ __device__ __forceinline__ void gemm_tc_store32(const GemmTcParams& p, int64_t r
   } else if (!gemm_epi_is_glu(p.epi)) {
     float a[32];
 #pragma unroll
-    for (int i = 0; i < 32; ++i) a[i] = gemm_store_act(v[i], p.epi, p.act);
+    for (int i = 0; i < 32; ++i) a[i] = v[i];
+    if (p.epi == B200P_GEMM_XIELU) {               // one uniform branch for all elements
+#pragma unroll
+      for (int i = 0; i < 32; ++i) a[i] = xielu_unit(v[i], p.act);
+    } else if (p.epi != B200P_GEMM_STORE) {
+#pragma unroll
+      for (int i = 0; i < 32; ++i) a[i] = gemm_store_act(v[i], p.epi, p.act);
+    }
     T* dst = reinterpret_cast<T*>(p.y) + row_off + n0;
     if (p.vec_ok && n0 + 32 <= p.N) {
 #pragma unroll
