@@ -274,7 +274,8 @@ enum {
   B200P_GEMM_GLU_GELU_TANH = 3, /* same row pairs: y = gelu_tanh(gate) * up                                          */
   B200P_GEMM_GLU_SILU = 4,   /* same row pairs: y = gate * sigmoid(gate) * up                                       */
   B200P_GEMM_RELU_SQ = 5,    /* y[M,N] (dtype) = max(acc, 0)^2: the hidden units of an ungated feed-forward           */
-  B200P_GEMM_XIELU = 6       /* y[M,N] (dtype) = act_a z^2 + z / 2 (z > 0), act_b (e^z - 1 - z) + z / 2 (z <= 0), z = acc */
+  B200P_GEMM_XIELU = 6,      /* y[M,N] (dtype) = act_a z^2 + z / 2 (z > 0), act_b (e^z - 1 - z) + z / 2 (z <= 0), z = acc */
+  B200P_GEMM_CAP_F32 = 7     /* y[M,N] (float) = act_a tanh(acc / act_a): capped logits                              */
 };
 /* act_a / act_b: the epilogue's constants (0 where it has none).
  * y = x . w^T, x [M,K] and w [N,K] in `dtype` (row strides ldx / ldw elements), fp32 accumulation; `batch` independent
@@ -321,10 +322,12 @@ int b200p_embed_hashed(const int32_t* ids, const int32_t* t_row, const int32_t* 
 int b200p_norm_add_norm(const float* y, const float* w_post, float* h, const float* w_next, void* x_out, void* raw_out,
                         int64_t M, int64_t W, float eps, int dtype, void* stream);
 /* Residual stream of designs that add their sublayers without a norm of their own, one pass per row:
- *   h += c1 * y1 + c2 * y2 (either may be NULL);  raw_out (rows of stride ld_raw) = h in `dtype`;
- *   x_out = h / sqrt(mean(h^2) + eps) * w_next in `dtype`.  rows [M, W]; h, y, weights fp32. */
-int b200p_residual_add_norm(float* h, const float* y1, float c1, const float* y2, float c2, const float* w_next, void* x_out,
-                            void* raw_out, int64_t ld_raw, int64_t M, int64_t W, float eps, int dtype, void* stream);
+ *   h += c1 * s1 y1 + c2 * s2 y2 (either y may be NULL; s1, s2 [W] scale channel by channel, NULL: ones);
+ *   raw_out (rows of stride ld_raw) = h in `dtype`;  x_out = h / sqrt(mean(h^2) + eps) * w_next in `dtype`;
+ *   x_out2 = the same unit row * w_next2 (a second reader's norm; NULL: none).  rows [M, W]; h, y, weights fp32. */
+int b200p_residual_add_norm(float* h, const float* y1, float c1, const float* s1, const float* y2, float c2, const float* s2,
+                            const float* w_next, void* x_out, const float* w_next2, void* x_out2, void* raw_out, int64_t ld_raw, int64_t M,
+                            int64_t W, float eps, int dtype, void* stream);
 /* dst[t, c] (dtype, row stride ld_dst) = src[t, c] (fp32, row stride ld_src), c < n */
 int b200p_cast_columns(const float* src, int64_t ld_src, void* dst, int64_t ld_dst, int64_t M, int64_t n, int dtype, void* stream);
 /* out[t, c] (dtype) = gelu_tanh(gate[t, c]) * table[ids[t], col0 + c], c < d; gate fp32 [M, d], table [*, ld_table] `dtype` */
@@ -405,9 +408,11 @@ int b200p_moe_route_sigmoid(const float* logits, int64_t ldl, const float* corre
                             int32_t* slot_of, int32_t* token_of, int64_t M, int E, int top, int count, int keep, float scale,
                             void* stream);
 /* The same outputs from plain scores: the `top` largest s = sigmoid(logits), or (softmax != 0) s = softmax(logits) over all
- * experts, are picked (ties to the smaller index) and wts are those scores as they are, not renormalised. */
+ * experts, are picked (ties to the smaller index) among the experts of the `keep` best of `count` equal groups of neighbouring
+ * experts (here a group's score = its LARGEST score; count == 1 or keep == count: no group limit); wts are those scores as they
+ * are, or (renorm != 0) divided by their sum (+ 1e-20). */
 int b200p_moe_route_scores(const float* logits, int64_t ldl, int32_t* ids, float* wts, int32_t* seg, int32_t* slot_of,
-                           int32_t* token_of, int64_t M, int E, int top, int softmax, void* stream);
+                           int32_t* token_of, int64_t M, int E, int top, int softmax, int count, int keep, int renorm, void* stream);
 /* Residual step of designs whose sublayers are normed on their output only, with an optional weighted sum over the embedding
  * output and all layers' results ("depth average").  Per token, fp32: x = h + rms_norm(y) w (y NULL: x = rms_norm(h) w);
  * stack[t, slot] = x (slot >= 0; stack [M, slots, W]); h = sum_{j < n-1} a[j] stack[t, j] + a[n-1] x (a NULL: h = x);
@@ -415,16 +420,20 @@ int b200p_moe_route_scores(const float* logits, int64_t ldl, int32_t* ids, float
 int b200p_post_norm_step(const float* y, const float* w, float* h, float* stack, int64_t slots, int slot, const float* a, int n,
                          void* raw_out, int64_t M, int64_t W, float eps, int dtype, void* stream);
 
-/* Attention whose heads' scores are mixed by a matrix before the softmax.  Preparation: proj columns [q | k | v] plus `bias`
- * (indexed by the same columns; NULL: none); q and k rms-normed over their WHOLE rows with weights wq [H dk] / wk [G dk] (NULL: not
- * normed); the first 2 n_rot dimensions of every head rotated by position * rates[i], cos and sin times `mag`, dimension i paired
- * with i + n_rot (pairs 0) or 2i with 2i + 1 (pairs 1); q_out [M, H dk] fp32 = q * scale; k, v into the caches
- * [rows, G, Tcap, dk] / [rows, G, Tcap, dv] at (t_row, t_pos). */
-int b200p_mix_attn_prep(const float* proj, int64_t ldp, int64_t col_q, int64_t col_k, int64_t col_v, const float* bias, const float* wq,
-                        const float* wk, float eps, const float* rates, int n_rot, float mag, int pairs, float scale, float* q_out,
-                        void* kcache, void* vcache, int64_t Tcap, const int32_t* t_row, const int32_t* t_pos, int64_t M, int H, int G,
-                        int dk, int dv, int dtype, void* stream);
-/* out[t, h] = softmax_j(sum_g talk[h, g] q_g . k_j) v_j over 0 <= position - j < window (0: every j <= position), the denominator
+/* Preparation of grouped attention on biased projections with whole-row norms: proj columns [q | k | v] plus `bias` (indexed by the
+ * same columns; NULL: none); q and k rms-normed over their WHOLE rows with weights wq [H dk] / wk [G dk] (NULL: not normed); the
+ * first 2 n_rot dimensions of every head rotated by position * rates[i], cos and sin times `mag`, dimension i paired with i + n_rot
+ * (pairs 0) or 2i with 2i + 1 (pairs 1); q_out [M, H dk] fp32 = q * scale * (1 + temp_coef ln(floor((p + 1) / temp_every) + 1))
+ * (temp_coef 0: no temperature); v <- (1 - v_lambda) v + v_lambda v_first (fp32 [M, G dv], the same tokens' values of an earlier
+ * layer; NULL: not blended), left in v_keep (fp32 [M, G dv]) when given; k, v into the caches [rows, G, Tcap, dk] /
+ * [rows, G, Tcap, dv] at (t_row, t_pos). */
+int b200p_row_attn_prep(const float* proj, int64_t ldp, int64_t col_q, int64_t col_k, int64_t col_v, const float* bias, const float* wq,
+                        const float* wk, float eps, const float* rates, int n_rot, float mag, int pairs, float scale, float temp_coef,
+                        float temp_every, const float* v_first, float v_lambda, float* v_keep, float* q_out, void* kcache, void* vcache,
+                        int64_t Tcap, const int32_t* t_row, const int32_t* t_pos, int64_t M, int H, int G, int dk, int dv, int dtype,
+                        void* stream);
+/* Attention whose heads' scores are mixed by a matrix before the softmax:
+ * out[t, h] = softmax_j(sum_g talk[h, g] q_g . k_j) v_j over 0 <= position - j < window (0: every j <= position), the denominator
  * also holding exp(sink[h]) (NULL: no sink).  talk fp32 [H, H]; 16-bit calls need talk exact in 11 significant bits (as a matrix
  * stored in 16 bits is).  Prompts of 16-bit models (key and value sizes 64 / 128, up to 16 heads, or up to 32 whose key heads serve
  * an even number) run on the tile kernel; the rest on the per-token kernel, whose decode steps (max_n 1) split the keys over CTAs

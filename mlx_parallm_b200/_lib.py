@@ -79,7 +79,7 @@ SIGNATURES = {
     "b200p_delta_out": (_i32, [_vp, _vp, _i64, _vp, _vp, _i64, _i64, _i32, _i32, _f32, _i32, _f32, _i32, _vp]),
     "b200p_linear_attn_prep": (_i32, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _vp]),
     "b200p_gemm_grouped": (_i32, [_vp, _vp, _vp, _vp, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i64, _i32, _i32, _f32, _f32, _vp]),
-    "b200p_residual_add_norm": (_i32, [_vp, _vp, _f32, _vp, _f32, _vp, _vp, _vp, _i64, _i64, _i64, _f32, _i32, _vp]),
+    "b200p_residual_add_norm": (_i32, [_vp, _vp, _f32, _vp, _vp, _f32, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i64, _f32, _i32, _vp]),
     "b200p_cast_columns": (_i32, [_vp, _i64, _vp, _i64, _i64, _i64, _i32, _vp]),
     "b200p_sink_attn_prep": (_i32, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _f32, _f32, _f32, _f32, _vp, _vp, _vp, _i64, _vp, _vp,
                                     _i64, _i32, _i32, _i32, _i32, _i32, _vp]),
@@ -91,7 +91,7 @@ SIGNATURES = {
     "b200p_moe_gather": (_i32, [_vp, _vp, _vp, _i64, _i64, _i32, _vp]),
     "b200p_moe_route_sigmoid": (_i32, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _f32, _vp]),
     "b200p_moe_combine": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _vp, _i64, _i64, _i32, _vp]),
-    "b200p_moe_route_scores": (_i32, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _vp]),
+    "b200p_moe_route_scores": (_i32, [_vp, _i64, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _i32, _i32, _vp]),
     "b200p_moe_scatter_scaled": (_i32, [_vp, _vp, _vp, _vp, _i64, _i64, _i32, _i32, _vp]),
     "b200p_ssm_prep": (_i32, [_vp, _i64, _i64, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i32, _i32,
                               _i32, _i32, _i32, _vp]),
@@ -121,8 +121,8 @@ SIGNATURES = {
     "b200p_canon_conv": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _i32, _i32, _vp]),
     "b200p_tanh_norm": (_i32, [_vp, _vp, _vp, _vp, _vp, _i64, _i64, _i32, _vp]),
     "b200p_post_norm_step": (_i32, [_vp, _vp, _vp, _vp, _i64, _i32, _vp, _i32, _vp, _i64, _i64, _f32, _i32, _vp]),
-    "b200p_mix_attn_prep": (_i32, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _f32, _vp, _i32, _f32, _i32, _f32, _vp, _vp, _vp, _i64, _vp,
-                                   _vp, _i64, _i32, _i32, _i32, _i32, _i32, _vp]),
+    "b200p_row_attn_prep": (_i32, [_vp, _i64, _i64, _i64, _i64, _vp, _vp, _vp, _f32, _vp, _i32, _f32, _i32, _f32, _f32, _f32, _vp, _f32, _vp,
+                                   _vp, _vp, _vp, _i64, _vp, _vp, _i64, _i32, _i32, _i32, _i32, _i32, _vp]),
     "b200p_mix_attn": (_i32, [_vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _i32, _i32, _vp, _vp, _i64, _vp, _i64, _i64, _i32, _i32, _i32, _i32,
                               _i32, _vp, _sz, _vp]),
     "b200p_mix_attn_workspace_bytes": (_sz, [_i64, _i32, _i32]),
@@ -137,14 +137,22 @@ UNIT_SETS = {
     "sequence_ssm": ("runtime", "dense_gemm", "dense_gemm_tc", "ragged", "delta_rule", "ssm", "diff_attn", "moe", "sampler"),
     "sequence_hyper": ("runtime", "dense_gemm", "dense_gemm_tc", "ragged", "hyper", "delta_rule", "latent_attn", "sink_attn", "moe",
                        "sampler"),
-    "sequence_post": ("runtime", "dense_gemm", "dense_gemm_tc", "ragged", "post_norm", "latent_attn", "mix_attn", "moe", "sampler"),
+    "sequence_post": ("runtime", "dense_gemm", "dense_gemm_tc", "ragged", "post_norm", "latent_attn", "row_attn_prep", "mix_attn", "moe",
+                      "sampler"),
+    "sequence_rows": ("runtime", "dense_gemm", "dense_gemm_tc", "ragged", "row_attn_prep", "sink_attn", "moe", "sampler"),
 }
-GEMM_STORE, GEMM_STORE_F32, GEMM_GLU_CLAMP, GEMM_GLU_GELU_TANH, GEMM_GLU_SILU, GEMM_RELU_SQ, GEMM_XIELU = 0, 1, 2, 3, 4, 5, 6
+GEMM_STORE, GEMM_STORE_F32, GEMM_GLU_CLAMP, GEMM_GLU_GELU_TANH, GEMM_GLU_SILU, GEMM_RELU_SQ, GEMM_XIELU, GEMM_CAP_F32 = 0, 1, 2, 3, 4, 5, 6, 7
 
 
 def gemm_is_gated(epilogue: int) -> bool:
     """Epilogues that read (gate, up) row pairs and write half as many columns."""
     return GEMM_GLU_CLAMP <= epilogue <= GEMM_GLU_SILU
+
+
+def gemm_is_f32(epilogue: int) -> bool:
+    """Epilogues that write float32 whatever the operands' type."""
+    return epilogue in (GEMM_STORE_F32, GEMM_CAP_F32)
+
 
 SCAN_DELTA, SCAN_DELTA_CHANNEL, SCAN_ACCUMULATE = 0, 1, 2
 GATE_SILU, GATE_SIGMOID = 0, 1

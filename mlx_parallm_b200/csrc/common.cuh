@@ -95,6 +95,11 @@ __device__ __forceinline__ float gemm_store_act(float v, int epi, float2 act) {
   if (epi == B200P_GEMM_XIELU) return xielu_unit(v, act);
   return v;
 }
+// epilogues that write fp32: the accumulator itself, or capped to (-cap, cap) by a tanh
+__device__ __forceinline__ bool gemm_epi_is_f32(int epi) { return epi == B200P_GEMM_STORE_F32 || epi == B200P_GEMM_CAP_F32; }
+__device__ __forceinline__ float gemm_f32_act(float v, int epi, float2 act) {
+  return epi == B200P_GEMM_CAP_F32 ? act.x * tanhf(v / act.x) : v;
+}
 __device__ __forceinline__ float glu_unit(float gate, float up, int epi, float2 act) {
   if (epi == B200P_GEMM_GLU_CLAMP) {
     const float limit = act.x;

@@ -30,10 +30,10 @@ static int g_gemm_path = 0;
 template <typename T>
 __device__ __forceinline__ void gemm_store_pair(void* y, int64_t row_off, int64_t n, int64_t N, float v0, float v1, int epi,
                                                 float2 act) {
-  if (epi == B200P_GEMM_STORE_F32) {
+  if (gemm_epi_is_f32(epi)) {
     float* p = reinterpret_cast<float*>(y) + row_off;
-    if (n < N) p[n] = v0;
-    if (n + 1 < N) p[n + 1] = v1;
+    if (n < N) p[n] = gemm_f32_act(v0, epi, act);
+    if (n + 1 < N) p[n + 1] = gemm_f32_act(v1, epi, act);
   } else if (!gemm_epi_is_glu(epi)) {
     T* p = reinterpret_cast<T*>(y) + row_off;
     if (n < N) p[n] = Tr<T>::from_f(gemm_store_act(v0, epi, act));
@@ -435,7 +435,8 @@ extern "C" int b200p_gemm_grouped(const void* x, const void* w, void* y, const i
   B200P_REQUIRE(x && w && y && seg, B200P_ERR_ARG, "null pointer");
   B200P_REQUIRE(total_rows >= max_rows, B200P_ERR_ARG, "x has fewer rows than a group may have");
   B200P_REQUIRE(max_rows >= 0 && N > 0 && K > 0 && groups > 0 && groups < 65536 && ldx >= K && ldw >= K, B200P_ERR_ARG, "bad GEMM shape");
-  B200P_REQUIRE(epilogue >= B200P_GEMM_STORE && epilogue <= B200P_GEMM_XIELU, B200P_ERR_ARG, "unknown epilogue %d", epilogue);
+  B200P_REQUIRE(epilogue >= B200P_GEMM_STORE && epilogue <= B200P_GEMM_CAP_F32, B200P_ERR_ARG, "unknown epilogue %d", epilogue);
+  B200P_REQUIRE(epilogue != B200P_GEMM_CAP_F32 || act_a > 0.f, B200P_ERR_ARG, "the capped epilogue needs a positive cap");
   B200P_REQUIRE(epilogue < B200P_GEMM_GLU_CLAMP || epilogue > B200P_GEMM_GLU_SILU || N % 2 == 0, B200P_ERR_ARG, "the gated epilogue needs gate / up row pairs");
   B200P_REQUIRE((max_rows + 63) / 64 < 65536, B200P_ERR_ARG, "grid too large");
   if (max_rows == 0) return B200P_OK;
@@ -467,7 +468,8 @@ extern "C" int b200p_gemm(const void* x, const void* w, void* y, int64_t M, int6
   using namespace b200p;
   B200P_REQUIRE(x && w && y, B200P_ERR_ARG, "null pointer");
   B200P_REQUIRE(M >= 0 && N > 0 && K > 0 && batch > 0 && ldx >= K && ldw >= K, B200P_ERR_ARG, "bad GEMM shape");
-  B200P_REQUIRE(epilogue >= B200P_GEMM_STORE && epilogue <= B200P_GEMM_XIELU, B200P_ERR_ARG, "unknown epilogue %d", epilogue);
+  B200P_REQUIRE(epilogue >= B200P_GEMM_STORE && epilogue <= B200P_GEMM_CAP_F32, B200P_ERR_ARG, "unknown epilogue %d", epilogue);
+  B200P_REQUIRE(epilogue != B200P_GEMM_CAP_F32 || act_a > 0.f, B200P_ERR_ARG, "the capped epilogue needs a positive cap");
   B200P_REQUIRE(epilogue < B200P_GEMM_GLU_CLAMP || epilogue > B200P_GEMM_GLU_SILU || N % 2 == 0, B200P_ERR_ARG, "the gated epilogue needs gate / up row pairs");
   B200P_REQUIRE((M + 63) / 64 < 65536 && batch < 65536, B200P_ERR_ARG, "grid too large");
   if (M == 0) return B200P_OK;

@@ -86,7 +86,12 @@ template <> __device__ __forceinline__ uint32_t pack2<__nv_bfloat16>(float a, fl
 // 32 consecutive accumulator columns of one token row -> y
 template <typename T>
 __device__ __forceinline__ void gemm_tc_store32(const GemmTcParams& p, int64_t row_off, int64_t n0, const float (&v)[32]) {
-  if (p.epi == B200P_GEMM_STORE_F32) {
+  if (p.epi == B200P_GEMM_CAP_F32) {
+    float* dst = reinterpret_cast<float*>(p.y) + row_off + n0;
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      if (n0 + i < p.N) dst[i] = gemm_f32_act(v[i], p.epi, p.act);
+  } else if (p.epi == B200P_GEMM_STORE_F32) {
     float* dst = reinterpret_cast<float*>(p.y) + row_off + n0;
     if (p.vec_ok && n0 + 32 <= p.N) {
 #pragma unroll
@@ -171,6 +176,11 @@ __device__ __forceinline__ void gemm_tc_store32_trans(const GemmTcParams& p, int
       for (int i = 0; i < 32; ++i)
         if (tok0 + i < p.N) dst[(tok0 + i) * p.ldy] = v[i];
     }
+  } else if (p.epi == B200P_GEMM_CAP_F32) {
+    float* dst = reinterpret_cast<float*>(p.y) + z_off + n;
+#pragma unroll
+    for (int i = 0; i < 32; ++i)
+      if (tok0 + i < p.N) dst[(tok0 + i) * p.ldy] = gemm_f32_act(v[i], p.epi, p.act);
   } else {
     T* dst = reinterpret_cast<T*>(p.y) + z_off + n;
 #pragma unroll
@@ -466,7 +476,7 @@ int gemm_tc_launch(const T* x, const T* w, void* y, int64_t M, int64_t N, int64_
   p.groups = 0;
   p.epi = epi;
   p.act = act;
-  const int64_t eb = epi == B200P_GEMM_STORE_F32 ? 4 : 2;
+  const int64_t eb = (epi == B200P_GEMM_STORE_F32 || epi == B200P_GEMM_CAP_F32) ? 4 : 2;
   p.vec_ok = aligned(y, 16) && (ldy * eb) % 16 == 0 && (sy * eb) % 16 == 0;
   if (bn == 256) return gemm_tc_run<T, 256, 4>(tmx, tmw, p, st);
   if (bn == 128) return gemm_tc_run<T, 128, 6>(tmx, tmw, p, st);
@@ -505,7 +515,7 @@ int gemm_tc_launch_grouped(const T* x, const T* w, void* y, const int32_t* seg, 
   p.groups = (int)groups;
   p.epi = epi;
   p.act = act;
-  const int64_t eb = epi == B200P_GEMM_STORE_F32 ? 4 : 2;
+  const int64_t eb = (epi == B200P_GEMM_STORE_F32 || epi == B200P_GEMM_CAP_F32) ? 4 : 2;
   p.vec_ok = aligned(y, 16) && (ldy * eb) % 16 == 0;
   if (bn == 256) return gemm_tc_run<T, 256, 4>(tmx, tmw, p, st);
   if (bn == 128) return gemm_tc_run<T, 128, 6>(tmx, tmw, p, st);

@@ -1,8 +1,8 @@
 // Routed mixture of experts over a packed token batch:
 //   moe_route_kernel    fp32 router logits (+ bias) -> the `top` largest per token and the softmax over those alone   (per token)
-//   moe_route_sigmoid_kernel  scores = sigmoid(logits); experts picked by score + correction inside the best expert groups;
-//                       weights = the picked experts' scores over their sum, times a scale; or the scores as they are, of
-//                       sigmoids or of a softmax over all experts                                                       (per token)
+//   moe_route_scores_kernel  scores = sigmoid(logits), or their softmax over all experts; experts picked by score (+ correction)
+//                       inside the best expert groups, a group counting as its best expert or as the sum of its two best; weights =
+//                       the picked experts' scores over their sum, times a scale, or the scores as they are              (per token)
 //   moe_plan_kernel     tokens counted per expert, segment offsets, a slot for every (token, choice)                 (one CTA)
 //   moe_gather_kernel   activation rows copied into slot order, so that an expert's rows are contiguous              (per slot)
 //   moe_combine_kernel  y[t] = gate[t] shared[t] + sum_k weight[t, k] * expert_out[slot(t, k)], in the order of the choices   (per token)
@@ -55,12 +55,13 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int64_t ldl, 
 }
 
 // One warp per token.  s_e = sigmoid(z_e); picking score c_e = s_e + correction_e.  The experts form `count` groups of
-// neighbours; a group's score is the sum of its two largest picking scores (its only one for groups of one expert); only the
-// experts of the `keep` best groups can be picked (the others count as -inf, since picking scores may be negative).  The `top`
-// largest picking scores win, ties to the smaller index; weights w_k = s_k / (sum of the picked s + 1e-20) * scale.
-__global__ void moe_route_sigmoid_kernel(const float* __restrict__ logits, int64_t ldl, const float* __restrict__ correction,
+// neighbours; a group's score is the sum of its two largest picking scores (its only one for groups of one expert), or (group_best)
+// its largest; only the experts of the `keep` best groups can be picked (the others count as -inf, since picking scores may be
+// negative).  The `top` largest picking scores win, ties to the smaller index; weights w_k = s_k / (sum of the picked s + 1e-20) *
+// scale.  softmax: s = softmax(z) over ALL experts, picked (and groups compared) by z, which orders the experts as s does.
+__global__ void moe_route_scores_kernel(const float* __restrict__ logits, int64_t ldl, const float* __restrict__ correction,
                                          int32_t* __restrict__ ids, float* __restrict__ wts, int64_t M, int E, int top, int count,
-                                         int keep, float scale, int renorm, int softmax) {
+                                         int keep, float scale, int renorm, int softmax, int group_best) {
   extern __shared__ float mr_sm[];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int64_t t = (int64_t)blockIdx.x * (blockDim.x >> 5) + warp;
@@ -97,7 +98,7 @@ __global__ void moe_route_sigmoid_kernel(const float* __restrict__ logits, int64
         if (v > a) { b = a; a = v; }
         else if (v > b) b = v;
       }
-      gs[g] = per > 1 ? a + b : a;
+      gs[g] = per > 1 && !group_best ? a + b : a;
     }
     __syncwarp();
     // drop the count - keep worst groups: repeatedly the smallest score, ties dropping the larger index first
@@ -259,33 +260,36 @@ extern "C" int b200p_moe_route_sigmoid(const float* logits, int64_t ldl, const f
   const int warps = 4;
   const size_t smem = (size_t)warps * (2 * E + count) * sizeof(float);
   if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(moe_route_sigmoid_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return cuda_fail(e, "cudaFuncSetAttribute(moe_route_sigmoid_kernel)");
+    cudaError_t e = cudaFuncSetAttribute(moe_route_scores_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return cuda_fail(e, "cudaFuncSetAttribute(moe_route_scores_kernel)");
   }
-  moe_route_sigmoid_kernel<<<(unsigned)((M + warps - 1) / warps), warps * 32, smem, st>>>(logits, ldl, correction, ids, wts, M, E, top,
-                                                                                           count, keep, scale, 1, 0);
-  B200P_LAUNCH_CHECK("moe_route_sigmoid_kernel");
+  moe_route_scores_kernel<<<(unsigned)((M + warps - 1) / warps), warps * 32, smem, st>>>(logits, ldl, correction, ids, wts, M, E, top,
+                                                                                           count, keep, scale, 1, 0, 0);
+  B200P_LAUNCH_CHECK("moe_route_scores_kernel");
   moe_plan_kernel<<<1, 1024, 2 * E * sizeof(int32_t), st>>>(ids, seg, slot_of, token_of, M * top, E, top);
   B200P_LAUNCH_CHECK("moe_plan_kernel");
   return B200P_OK;
 }
 
 extern "C" int b200p_moe_route_scores(const float* logits, int64_t ldl, int32_t* ids, float* wts, int32_t* seg, int32_t* slot_of,
-                                      int32_t* token_of, int64_t M, int E, int top, int softmax, void* stream) {
+                                      int32_t* token_of, int64_t M, int E, int top, int softmax, int count, int keep, int renorm,
+                                      void* stream) {
   B200P_REQUIRE(logits && ids && wts && seg && slot_of && token_of, B200P_ERR_ARG, "null pointer");
   B200P_REQUIRE(E > 0 && E <= 32 * MOE_MAX_PER_LANE && top > 0 && top <= E && top <= MOE_MAX_TOP, B200P_ERR_ARG,
                 "experts in [1, %d] and top in [1, min(experts, %d)]", 32 * MOE_MAX_PER_LANE, MOE_MAX_TOP);
+  B200P_REQUIRE(count >= 1 && E % count == 0 && keep >= 1 && keep <= count && (int64_t)keep * (E / count) >= top, B200P_ERR_ARG,
+                "expert groups: equal groups, 1 <= keep <= count, and the kept groups hold at least `top` experts");
   if (M == 0) return B200P_OK;
   cudaStream_t st = (cudaStream_t)stream;
   const int warps = 4;
-  const size_t smem = (size_t)warps * (2 * E + 1) * sizeof(float);
+  const size_t smem = (size_t)warps * (2 * E + count) * sizeof(float);
   if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(moe_route_sigmoid_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return cuda_fail(e, "cudaFuncSetAttribute(moe_route_sigmoid_kernel)");
+    cudaError_t e = cudaFuncSetAttribute(moe_route_scores_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return cuda_fail(e, "cudaFuncSetAttribute(moe_route_scores_kernel)");
   }
-  moe_route_sigmoid_kernel<<<(unsigned)((M + warps - 1) / warps), warps * 32, smem, st>>>(logits, ldl, nullptr, ids, wts, M, E, top, 1, 1,
-                                                                                           1.f, 0, softmax);
-  B200P_LAUNCH_CHECK("moe_route_sigmoid_kernel");
+  moe_route_scores_kernel<<<(unsigned)((M + warps - 1) / warps), warps * 32, smem, st>>>(logits, ldl, nullptr, ids, wts, M, E, top,
+                                                                                          count, keep, 1.f, renorm, softmax, 1);
+  B200P_LAUNCH_CHECK("moe_route_scores_kernel");
   moe_plan_kernel<<<1, 1024, 2 * E * sizeof(int32_t), st>>>(ids, seg, slot_of, token_of, M * top, E, top);
   B200P_LAUNCH_CHECK("moe_plan_kernel");
   return B200P_OK;

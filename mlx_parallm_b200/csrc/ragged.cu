@@ -112,32 +112,114 @@ __global__ void norm_add_norm_kernel(const float* __restrict__ y, const float* _
   }
 }
 
-// Residual stream of designs whose sublayers are added without a norm of their own (several branches may read one normed
-// input and are summed into the stream together): h += c1 y1 + c2 y2, then the copies the next step needs.
-template <typename T>
-__global__ void residual_add_norm_kernel(float* __restrict__ h, const float* __restrict__ y1, float c1, const float* __restrict__ y2,
-                                         float c2, const float* __restrict__ w_next, T* __restrict__ x_out, T* __restrict__ raw_out,
-                                         int64_t ld_raw, int64_t W, float eps) {
-  __shared__ float red[32];
-  const int64_t row = blockIdx.x;
-  float* hr = h + row * W;
-  float hs = 0.f;
-  for (int64_t c = threadIdx.x; c < W; c += blockDim.x) {
-    float v = hr[c];
-    if (y1 || y2) {
-      float add = 0.f;
-      if (y1) add = c1 * y1[row * W + c];
-      if (y2) add += c2 * y2[row * W + c];
-      v += add;
-      hr[c] = v;
-    }
-    hs = fmaf(v, v, hs);
-    if (raw_out) raw_out[row * ld_raw + c] = Tr<T>::from_f(v);
+// Residual stream of designs whose sublayers are added without a norm of their own (several branches may be summed into the stream
+// together, each scaled channel by channel): h += c1 s1 y1 + c2 s2 y2, then the copies the next step needs: the row in the storage
+// type and up to two normed versions of it (two readers with norms of their own share the root mean square).
+struct ResidualOut {
+  const float* w1;       // weights of x1 / x2
+  const float* w2;
+  void* x1;
+  void* x2;
+  void* raw;
+  int64_t ld_raw;
+};
+
+template <typename T, int V>
+__device__ __forceinline__ void store_row(T* d, const float (&v)[V]) {
+  if constexpr (V == 4 && sizeof(T) == 2) {
+    __align__(8) T o[4] = {Tr<T>::from_f(v[0]), Tr<T>::from_f(v[1]), Tr<T>::from_f(v[2]), Tr<T>::from_f(v[3])};
+    *reinterpret_cast<uint2*>(d) = *reinterpret_cast<const uint2*>(o);
+  } else if constexpr (V == 4) {
+    *reinterpret_cast<float4*>(d) = make_float4(v[0], v[1], v[2], v[3]);
+  } else {
+    d[0] = Tr<T>::from_f(v[0]);
   }
-  if (x_out) {
-    hs = block_sum(hs, red);
-    const float invh = 1.f / sqrtf(hs / (float)W + eps);
-    for (int64_t c = threadIdx.x; c < W; c += blockDim.x) x_out[row * W + c] = Tr<T>::from_f(hr[c] * invh * w_next[c]);
+}
+template <int V>
+__device__ __forceinline__ void load_row(const float* p, float (&v)[V]) {
+  if constexpr (V == 4) {
+    const float4 q = *reinterpret_cast<const float4*>(p);
+    v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w;
+  } else {
+    v[0] = p[0];
+  }
+}
+
+// V neighbouring channels per access; the first R pieces of a thread's row stay in registers between the sum of squares and the
+// normed stores, longer rows are read again (by the thread that wrote them).
+template <typename T, int V, int R>
+__global__ void residual_add_norm_kernel(float* __restrict__ h, const float* __restrict__ y1, float c1, const float* __restrict__ s1,
+                                         const float* __restrict__ y2, float c2, const float* __restrict__ s2, ResidualOut out, int64_t W,
+                                         float eps) {
+  __shared__ float red[32];
+  const int64_t row = blockIdx.x, step = (int64_t)blockDim.x * V;
+  float* hr = h + row * W;
+  T* raw = reinterpret_cast<T*>(out.raw);
+  T* x1 = reinterpret_cast<T*>(out.x1);
+  T* x2 = reinterpret_cast<T*>(out.x2);
+  float hs = 0.f;
+  float keep[R][V];
+  auto piece = [&](int64_t c, float (&v)[V]) {
+    load_row<V>(hr + c, v);
+    if (y1 || y2) {
+      float add[V];
+#pragma unroll
+      for (int k = 0; k < V; ++k) add[k] = 0.f;
+      if (y1) {
+        float a[V], s[V];
+        load_row<V>(y1 + row * W + c, a);
+        if (s1) load_row<V>(s1 + c, s);
+#pragma unroll
+        for (int k = 0; k < V; ++k) add[k] = c1 * (s1 ? s[k] * a[k] : a[k]);
+      }
+      if (y2) {
+        float a[V], s[V];
+        load_row<V>(y2 + row * W + c, a);
+        if (s2) load_row<V>(s2 + c, s);
+#pragma unroll
+        for (int k = 0; k < V; ++k) add[k] += c2 * (s2 ? s[k] * a[k] : a[k]);
+      }
+#pragma unroll
+      for (int k = 0; k < V; ++k) v[k] += add[k];
+      store_row<float, V>(hr + c, v);
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) hs = fmaf(v[k], v[k], hs);
+    if (raw) store_row<T, V>(raw + row * out.ld_raw + c, v);
+  };
+  const int64_t c0 = (int64_t)threadIdx.x * V;
+#pragma unroll
+  for (int r = 0; r < R; ++r)
+    if (c0 + r * step < W) piece(c0 + r * step, keep[r]);
+  for (int64_t c = c0 + R * step; c < W; c += step) {
+    float v[V];
+    piece(c, v);
+  }
+  if (!x1 && !x2) return;
+  hs = block_sum(hs, red);
+  const float inv = 1.f / sqrtf(hs / (float)W + eps);
+  auto normed = [&](int64_t c, const float (&v)[V]) {
+    float w[V], o[V];
+    if (x1) {
+      load_row<V>(out.w1 + c, w);
+#pragma unroll
+      for (int k = 0; k < V; ++k) o[k] = v[k] * inv * w[k];
+      store_row<T, V>(x1 + row * W + c, o);
+    }
+    if (x2) {
+      load_row<V>(out.w2 + c, w);
+#pragma unroll
+      for (int k = 0; k < V; ++k) o[k] = v[k] * inv * w[k];
+      store_row<T, V>(x2 + row * W + c, o);
+    }
+  };
+#pragma unroll
+  for (int r = 0; r < R; ++r)
+    if (c0 + r * step < W) normed(c0 + r * step, keep[r]);
+  for (int64_t c = c0 + R * step; c < W; c += step) {
+    float v[V];
+    load_row<V>(hr + c, v);
+    normed(c, v);
   }
 }
 
@@ -213,16 +295,30 @@ extern "C" int b200p_norm_add_norm(const float* y, const float* w_post, float* h
   return B200P_OK;
 }
 
-extern "C" int b200p_residual_add_norm(float* h, const float* y1, float c1, const float* y2, float c2, const float* w_next,
-                                       void* x_out, void* raw_out, int64_t ld_raw, int64_t M, int64_t W, float eps, int dtype,
-                                       void* stream) {
+extern "C" int b200p_residual_add_norm(float* h, const float* y1, float c1, const float* s1, const float* y2, float c2, const float* s2,
+                                       const float* w_next, void* x_out, const float* w_next2, void* x_out2, void* raw_out, int64_t ld_raw,
+                                       int64_t M, int64_t W, float eps, int dtype, void* stream) {
   B200P_REQUIRE(h && W > 0, B200P_ERR_ARG, "null residual stream");
-  B200P_REQUIRE(!x_out || w_next, B200P_ERR_ARG, "x_out needs its norm weight");
+  B200P_REQUIRE((!x_out || w_next) && (!x_out2 || w_next2), B200P_ERR_ARG, "x_out needs its norm weight");
   B200P_REQUIRE(!raw_out || ld_raw >= W, B200P_ERR_ARG, "raw_out rows are shorter than the stream");
   if (M == 0) return B200P_OK;
-  const unsigned threads = W >= 2048 ? 512 : (W >= 512 ? 256 : 128);
-  B200P_DISPATCH_DTYPE(dtype, T, (residual_add_norm_kernel<T><<<(unsigned)M, threads, 0, (cudaStream_t)stream>>>(
-      h, y1, c1, y2, c2, w_next, (T*)x_out, (T*)raw_out, ld_raw, W, eps)));
+  const ResidualOut out = {w_next, w_next2, x_out, x_out2, raw_out, ld_raw};
+  cudaStream_t st = (cudaStream_t)stream;
+  const bool vec = W % 4 == 0 && ld_raw % 4 == 0 && aligned(h, 16) && aligned(y1, 16) && aligned(y2, 16) && aligned(s1, 16) &&
+                   aligned(s2, 16) && aligned(w_next, 16) && aligned(w_next2, 16) && aligned(x_out, 16) && aligned(x_out2, 16) &&
+                   aligned(raw_out, 16);
+#define RES_CASE(V_, R_, THREADS_)                                                                                          \
+  B200P_DISPATCH_DTYPE(dtype, T, (residual_add_norm_kernel<T, V_, R_><<<(unsigned)M, THREADS_, 0, st>>>(h, y1, c1, s1, y2, c2, s2, out, W, eps)))
+  if (!vec) {
+    RES_CASE(1, 4, W >= 2048 ? 512u : (W >= 512 ? 256u : 128u));
+  } else if (W <= 512) {
+    RES_CASE(4, 1, 128u);
+  } else if (W <= 2048) {
+    RES_CASE(4, 2, 256u);
+  } else {
+    RES_CASE(4, 2, 512u);
+  }
+#undef RES_CASE
   B200P_LAUNCH_CHECK("residual_add_norm_kernel");
   return B200P_OK;
 }

@@ -4,7 +4,7 @@
 // nothing to the output, so it only takes probability mass away from the keys.
 //   sink_attn_prep_kernel   norms, temperature and scale on q; normed k and v into the cache at (row, position)     (per token)
 //   sink_attn_kernel        one token x the query heads of one key/value head, fp32 throughout, any sizes           (per token)
-//   sink_attn_tile_kernel   16 query rows per warp on mma.sync over 64-key tiles: 64 tokens of a prompt for one head, or the
+//   sink_attn_tile_kernel   16 query rows per warp on mma.sync over 64-key tiles: 64 tokens of a prompt for one head, or up to 16
 //                           heads of a key/value head for one decoded token with the keys split over CTAs              (16-bit caches)
 //   attn_merge_kernel       the decode step's partial sums and the sink                                               (per token, head)
 // The softmax starts from the sink: running maximum = sink, running sum = 1 (the sink's own term), accumulator = 0; every key
@@ -227,13 +227,19 @@ __global__ void window_attn_prep_kernel(const float* __restrict__ proj, int64_t 
 // global -> shared with cp.async (two stages, XOR-swizzled 16-byte chunks, shared by the four warps); S = Q K^T and O += P V
 // run on mma.sync m16n8k16 with the fp32 online softmax in registers, in base-2 units: the distance bias is added to the
 // scores as -slope log2(e) (p - j), and the running maximum / sum start from the sink (max = sink log2(e), sum = 1).
+// Rows of whole 128-byte lines are swizzled over eight keys; rows of 64 or 192 bytes alternate between the halves of a line by
+// themselves and are swizzled over four pairs of keys inside a half: either way eight neighbouring keys meet all 32 banks once.
+template <int CHUNKS>
+__device__ __forceinline__ int tile_chunk(int key, int ch) {
+  return CHUNKS % 8 == 0 ? ch ^ (key & 7) : ch ^ ((key >> 1) & 3);
+}
 constexpr int ST_WARPS = 4, ST_THREADS = ST_WARPS * 32, ST_QT = 16 * ST_WARPS, ST_KT = 64, ST_STAGES = 2;
 
 // DECODE = false: 4 warps, rows = 64 consecutive tokens of entry blockIdx.z for head blockIdx.y (tile blockIdx.x of the entry).
-// DECODE = true: ONE warp per CTA; its 16 rows are the query heads of key/value head blockIdx.y for the single token of entry
-// blockIdx.z, and the CTA takes the blockIdx.x-th share of the key tiles (gridDim.x shares): it writes unnormalised partial
-// sums (o, running max, sum; no sink) that attn_merge_kernel (attn_merge.cuh) combines.  The keys are then read once for all heads of a
-// group, by many small CTAs at a time.
+// DECODE = true: ONE warp per CTA; its 16 rows are query heads of one key/value head (blockIdx.y: key/value head x block of 16 of its
+// heads) for the single token of entry blockIdx.z, and the CTA takes the blockIdx.x-th share of the key tiles (gridDim.x shares): it
+// writes unnormalised partial sums (o, running max, sum; no sink) that attn_merge_kernel (attn_merge.cuh) combines.  The keys are then
+// read once for 16 heads of a group, by many small CTAs at a time.
 // RULED = true: the scores also pass the ScoreRule (cap, logarithmic penalty, window: tiles before the window of the CTA's first
 // row are skipped, a row whose window has not begun keeps max = -inf and adds nothing) and the output its gate.
 template <typename T, int DK, int DV, bool DECODE, bool RULED>
@@ -254,9 +260,10 @@ sink_attn_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc, con
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int quad_row = lane >> 2, qc = lane & 3;
   const int per = H / G;
-  const int g = DECODE ? blockIdx.y : blockIdx.y / per;
+  const int blocks = DECODE ? (per + 15) / 16 : 1;                  // blocks of 16 heads per key/value head
+  const int g = DECODE ? blockIdx.y / blocks : blockIdx.y / per;
   const int p_first = t_pos[t_first];                               // positions of an entry's tokens are consecutive
-  const int l0 = q0 + warp * 16 + quad_row, l1 = l0 + 8;            // this thread's two rows: tokens (prompts) or heads (decode)
+  const int l0 = (DECODE ? (blockIdx.y % blocks) * 16 : q0 + warp * 16) + quad_row, l1 = l0 + 8;     // this thread's two rows: tokens (prompts) or heads (decode)
   const int n_rows = DECODE ? per : n_e;
   const int lc0 = min(l0, n_rows - 1), lc1 = min(l1, n_rows - 1);   // rows past the end compute a valid row, not stored
   const int h0 = DECODE ? g * per + lc0 : blockIdx.y, h1 = DECODE ? g * per + lc1 : blockIdx.y;
@@ -316,7 +323,7 @@ sink_attn_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc, con
       const int idx = i * NT + threadIdx.x;
       const int key = idx / KCH, ch = idx % KCH;
       const bool ok = key0 + key < kend;
-      cp_async16(ks + (uint32_t)(key * KROW + ((ch ^ (key & 7)) << 4)), kbase + (int64_t)(key0 + (ok ? key : 0)) * DK + ch * 8, ok);
+      cp_async16(ks + (uint32_t)(key * KROW + (tile_chunk<KCH>(key, ch) << 4)), kbase + (int64_t)(key0 + (ok ? key : 0)) * DK + ch * 8, ok);
     }
     if (same_kv) return;
 #pragma unroll
@@ -324,7 +331,7 @@ sink_attn_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc, con
       const int idx = i * NT + threadIdx.x;
       const int key = idx / VCH, ch = idx % VCH;
       const bool ok = key0 + key < kend;
-      cp_async16(vs + (uint32_t)(key * VROW + ((ch ^ (key & 7)) << 4)), vbase + (int64_t)(key0 + (ok ? key : 0)) * DV + ch * 8, ok);
+      cp_async16(vs + (uint32_t)(key * VROW + (tile_chunk<VCH>(key, ch) << 4)), vbase + (int64_t)(key0 + (ok ? key : 0)) * DV + ch * 8, ok);
     }
   };
 
@@ -358,7 +365,7 @@ sink_attn_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc, con
       for (int kstep = 0; kstep < DK / 16; ++kstep) {
         const int ch = 2 * kstep + (mat & 1);
         uint32_t bf[4];
-        ldsm_x4(ks + (uint32_t)(key * KROW + ((ch ^ (key & 7)) << 4)), bf);
+        ldsm_x4(ks + (uint32_t)(key * KROW + (tile_chunk<KCH>(key, ch) << 4)), bf);
         mma16816<T>(sc[2 * np], qf[kstep], bf[0], bf[1]);
         mma16816<T>(sc[2 * np + 1], qf[kstep], bf[2], bf[3]);
       }
@@ -421,7 +428,7 @@ sink_attn_tile_kernel(const float* __restrict__ q, const T* __restrict__ kc, con
       for (int jp = 0; jp < DV / 16; ++jp) {
         const int ch = 2 * jp + (mat >> 1);
         uint32_t bf[4];
-        ldsm_x4_trans(vs + (uint32_t)(key * VROW + ((ch ^ (key & 7)) << 4)), bf);
+        ldsm_x4_trans(vs + (uint32_t)(key * VROW + (tile_chunk<VCH>(key, ch) << 4)), bf);
         mma16816<T>(o[2 * jp], pf, bf[0], bf[1]);
         mma16816<T>(o[2 * jp + 1], pf, bf[2], bf[3]);
       }
@@ -487,13 +494,14 @@ static int sink_attn_tiles_launch(const float* q, const void* kc, const void* vc
       attr_smem = smem;
     }
     const size_t per_split = (size_t)nb * H * (DV + 2) * sizeof(float);
-    int splits = (int)((8 * 148 + (int64_t)nb * G - 1) / ((int64_t)nb * G));
+    const int64_t work = (int64_t)nb * G * ((H / G + 15) / 16);
+    int splits = (int)((8 * 148 + work - 1) / work);
     splits = splits < 1 ? 1 : splits > SINK_ATTN_MAX_SPLITS ? SINK_ATTN_MAX_SPLITS : splits;
     if ((size_t)splits * per_split > ws_bytes) splits = (int)(ws_bytes / per_split);
     if (splits < 1) return 1;                                     // no room for partial sums: the caller takes the per-token kernel
     float* part_o = ws;
     float* part_ms = ws + (size_t)nb * H * splits * DV;
-    dim3 grid((unsigned)splits, (unsigned)G, (unsigned)nb);
+    dim3 grid((unsigned)splits, (unsigned)(work / nb), (unsigned)nb);
     kern<<<grid, 32, smem, st>>>(q, (const T*)kc, (const T*)vc, Tcap, cu, rows, t_pos, sink, slope_log2, (T*)out, ld_out, out_scale,
                                  H, G, part_o, part_ms, rule);
     B200P_LAUNCH_CHECK("sink_attn_tile_kernel");
@@ -516,9 +524,10 @@ static int sink_attn_tiles_launch(const float* q, const void* kc, const void* vc
   return B200P_OK;
 }
 
-// 1 when the tile kernel takes these sizes (16-bit caches, key and value sizes of 64 or 128)
+// 1 when the tile kernel takes these sizes (16-bit caches, key and value sizes of 32, 64, 96 or 128)
 static bool sink_attn_tiles_ok(int dk, int dv, int dtype) {
-  return (dtype == B200P_F16 || dtype == B200P_BF16) && (dk == 64 || dk == 128) && (dv == 64 || dv == 128);
+  auto size_ok = [](int d) { return d == 32 || d == 64 || d == 96 || d == 128; };
+  return (dtype == B200P_F16 || dtype == B200P_BF16) && size_ok(dk) && size_ok(dv);
 }
 
 template <typename T>
@@ -533,10 +542,12 @@ static int sink_attn_tiles(const float* q, const void* kc, const void* vc, int64
 #define ST_RULED(DK_, DV_) \
   if (dk == DK_ && dv == DV_ && rule) \
     return sink_attn_tiles_launch<T, DK_, DV_, true>(q, kc, vc, Tcap, cu, rows, t_pos, sink, slope_log2, out, ld_out, out_scale, nb, max_n, H, G, ws, ws_bytes, st, *rule)
-  ST_CASE(64, 64);
-  ST_CASE(64, 128);
-  ST_CASE(128, 64);
-  ST_CASE(128, 128);
+#define ST_VALUES(DK_) ST_CASE(DK_, 32); ST_CASE(DK_, 64); ST_CASE(DK_, 96); ST_CASE(DK_, 128)
+  ST_VALUES(32);
+  ST_VALUES(64);
+  ST_VALUES(96);
+  ST_VALUES(128);
+#undef ST_VALUES
   ST_RULED(64, 64);
   ST_RULED(128, 128);
   if (rule) return 1;                                            // other sizes with a rule: the caller takes the per-token kernel
@@ -604,9 +615,9 @@ static int attn_dispatch(const float* q, const void* kcache, const void* vcache,
   if (M == 0) return B200P_OK;
   cudaStream_t st = (cudaStream_t)stream;
   // prompts (entries of several tokens, described by cu / rows) of 16-bit models run on the tensor-core tile kernel
-  // and so do decode steps (one token per entry) whose heads per key/value head fit a 16-row tile, given room for partial sums
+  // and so do decode steps (one token per entry), given room for partial sums
   const bool prompts = max_n >= SINK_ATTN_TILES_MIN_TOKENS;
-  const bool decode = max_n == 1 && H / G <= 16 && workspace && aligned(workspace, 16);
+  const bool decode = max_n == 1 && workspace && aligned(workspace, 16);
   if (cu && rows && nb > 0 && (prompts || decode) && sink_attn_tiles_ok(dk, dv, dtype) && ld_out % 2 == 0 &&
       aligned(kcache, 16) && aligned(vcache, 16) && aligned(out, 4) && aligned(q, 8) && nb < 65536 && H < 65536) {
     const int rc = dtype == B200P_F16

@@ -22,22 +22,25 @@ layers mix a recurrent state with windowed attention over a shared low-rank late
     RoutedExperts           top-k routed GatedFF experts + a shared one; softmax     b200p_moe_* / b200p_gemm_grouped
                             over the chosen logits, sigmoid scores picked inside
                             the best expert groups with a gated shared expert, or
-                            plain sigmoid / softmax scores as they are
+                            plain sigmoid / softmax scores as they are or over
+                            their sum, with or without expert groups
     LatentAttention         queries and keys/values through low-rank latents,       b200p_latent_prep / b200p_latent_attn
                             sliding window, optional sharing of another layer's latents,  b200p_latent_rope_prep / _q_rope
                             optionally a rotated key part shared by the heads
-    HeadMixAttention        grouped-head attention whose heads' scores are mixed      b200p_mix_attn_prep / b200p_mix_attn
-                            by a matrix before the softmax: biases, q and k normed
-                            as whole rows, partial rotation, sliding window, sink
+    RowNormAttention        grouped-head attention, biases, q and k normed as whole   b200p_row_attn_prep / b200p_sink_attn
+                            rows, optional rotation, query temperature and sink,
+                            values blended with the first such layer's
+    HeadMixAttention        the same whose heads' scores are mixed by a matrix        b200p_row_attn_prep / b200p_mix_attn
+                            before the softmax: partial rotation, sliding window
     WindowAttention         grouped-head attention without rotation over a sliding    b200p_window_attn_prep / b200p_window_attn
                             window: short convolutions on q and k, values that are the
                             keys, capped scores, logarithmic distance penalty, output gate
     ClampedGLU              g * sigmoid(1.702 g) * (u + 1) on clamped gate / up      b200p_gemm (fused epilogue)
     TokenSideInput          a small per-layer table indexed by the token, gated      b200p_token_gate
     SequenceModel           the layer chain over a ragged batch: norm -> sublayer -> norm -> residual (b200p_norm_add_norm), or
-                            one norm feeding a mixer and a feed-forward that are added together, or a norm before each of the
-                            two, with an optional span of layers that runs several times on the same weights
-                            (b200p_residual_add_norm), or several copies of the stream that every sublayer reads as a weighted sum
+                            a mixer and a feed-forward that are added together (one norm for both or one each, optional scales
+                            per channel), or a norm before each of the two, with an optional span of layers that runs several
+                            times on the same weights (b200p_residual_add_norm), or several copies of the stream that every sublayer reads as a weighted sum
                             and writes back through a mixing matrix, with a tanh norm and a short convolution on what a sublayer
                             reads (b200p_hyper_step / b200p_canon_conv), or sublayers that read the stream itself and are normed on
                             their output only, with an optional weighted sum over all layers' results after every layer
@@ -59,8 +62,8 @@ import torch
 from .. import ops
 import math
 
-from .._lib import (GATE_SIGMOID, GATE_SILU, GEMM_GLU_CLAMP, GEMM_GLU_GELU_TANH, GEMM_GLU_SILU, GEMM_RELU_SQ, GEMM_STORE, GEMM_STORE_F32,
-                    GEMM_XIELU, SCAN_ACCUMULATE, SCAN_DELTA, SCAN_DELTA_CHANNEL)
+from .._lib import (GATE_SIGMOID, GATE_SILU, GEMM_CAP_F32, GEMM_GLU_CLAMP, GEMM_GLU_GELU_TANH, GEMM_GLU_SILU, GEMM_RELU_SQ, GEMM_STORE,
+                    GEMM_STORE_F32, GEMM_XIELU, SCAN_ACCUMULATE, SCAN_DELTA, SCAN_DELTA_CHANNEL)
 from .base import BatchedKVCache, ConvTailState, DeltaRuleState, LatentKVCache, RowState, StateGroup, TokenState
 
 MAX_TOKENS_PER_FORWARD = 8192     # packed tokens of one pass through the layers
@@ -621,54 +624,87 @@ class WindowAttention:
         return self.o_proj(mix, GEMM_STORE_F32, out=y_out)
 
 
-class HeadMixAttention:
+class RowNormAttention:
     """Causal attention with ``heads`` query heads over ``kv_heads`` key/value heads (query head h reads h // (heads // kv_heads)),
-    keys of ``dim`` and values of ``vdim``, whose heads' scores are mixed before the softmax:
-    score_h = sum_g talk[h, g] (q_g . k_g * scale).  q, k, v carry biases (``bias``); q and k are rms-normed over ALL their heads at
-    once (``row_norm``); the first 2 len(rates) dimensions of every head are rotated by position * rates[i], cos and sin times
-    ``mag``, dimension i paired with i + len(rates) (``pairs``: 2i with 2i + 1); ``window`` > 0: position i sees j with
-    0 <= i - j < window; the softmax denominator also holds exp(sink_h) (``sink`` False: not).  Projection columns [q | k | v]; the
-    rotated keys and the values are cached per position."""
+    keys of ``dim`` and values of ``vdim``.  q, k, v carry biases (``bias``); q and k are rms-normed over ALL their heads at once
+    (``row_norm``); the first 2 len(rates) dimensions of every head are rotated by position * rates[i], cos and sin times ``mag``,
+    dimension i paired with i + len(rates) (``pairs``: 2i with 2i + 1); q at position p is multiplied by
+    1 + temp_coef ln(floor((p + 1) / temp_every) + 1); score = q . k * scale; the softmax denominator also holds exp(sink_h)
+    (``sink`` False: not).  ``values``: "own"; "first" leaves the layer's values (fp32) for later layers of the same pass;
+    "blend" turns v into (1 - value_mix) v + value_mix v_first with the values that a "first" layer of equal sizes left.  Projection
+    columns [q | k | v]; the prepared keys and the values are cached per position."""
 
     DECODE_WS_ROWS = 256
 
     def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, rates: Sequence[float] = (),
-                 mag: float = 1.0, pairs: bool = False, window: int = 0, bias: bool = True, row_norm: bool = True, sink: bool = True):
+                 mag: float = 1.0, pairs: bool = False, bias: bool = True, row_norm: bool = True, sink: bool = False, temp_coef: float = 0.0,
+                 temp_every: float = 1.0, values: str = "own"):
         if heads % kv_heads or 2 * len(rates) > dim:
             raise ValueError("heads must be a multiple of kv_heads and the rotated dimensions at most dim")
+        if values not in ("own", "first", "blend"):
+            raise ValueError(f"unknown use of the values {values!r}")
         self.width, self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.eps = width, heads, kv_heads, dim, vdim, float(scale), eps
-        self.rate_values, self.mag, self.pairs, self.window = [float(r) for r in rates], float(mag), bool(pairs), int(window)
+        self.rate_values, self.mag, self.pairs = [float(r) for r in rates], float(mag), bool(pairs)
         self.has_bias, self.row_norm, self.has_sink = bool(bias), bool(row_norm), bool(sink)
+        self.temp_coef, self.temp_every, self.values = float(temp_coef), float(temp_every), values
+        self.value_mix = 0.0
         self.col_k = heads * dim
         self.col_v = self.col_k + kv_heads * dim
         self.n_proj = self.col_v + kv_heads * vdim
         self.n_mix = heads * vdim
         self.in_proj = Linear(width, self.n_proj)
         self.o_proj = Linear(self.n_mix, width)
-        self.bias = self.q_norm_w = self.k_norm_w = self.talk = self.sink = self.rates = None      # fp32 on the device
+        self.bias = self.q_norm_w = self.k_norm_w = self.sink = self.rates = None      # fp32 on the device
 
     def new_state(self, batch_size: int) -> RowState:
         return BatchedKVCache(self.dim, self.kv_heads, batch_size, value_dim=self.vdim)
+
+    def workspace_floats(self, rows: int) -> int:
+        return ops.sink_attn_workspace_floats(rows, self.heads, self.vdim)
 
     def reserve(self, s: Scratch, dt):
         s.reserve("proj", torch.float32, self.n_proj)
         s.reserve("aq", torch.float32, self.col_k)
         s.reserve("mix", dt, self.n_mix)
+        if self.values != "own":
+            s.reserve("v_first", torch.float32, self.kv_heads * self.vdim)
         if dt != torch.float32:
-            s.reserve_flat("attn_ws", torch.float32, ops.mix_attn_workspace_floats(min(s.rows, self.DECODE_WS_ROWS), self.heads, self.vdim))
+            s.reserve_flat("attn_ws", torch.float32, self.workspace_floats(min(s.rows, self.DECODE_WS_ROWS)))
+
+    def attend(self, q, st: BatchedKVCache, mix, plan: dict, workspace):
+        ops.sink_attn(q, st.keys, st.values, plan["t_row"], plan["t_pos"], self.sink, 0.0, mix, self.heads, self.kv_heads, self.dim, self.vdim,
+                      1.0, cu=plan["cu"], rows=plan["rows"], nb=plan["nb"], max_n=plan["max_n"], workspace=workspace)
 
     def __call__(self, x, y_out, st: BatchedKVCache, plan: dict, s: Scratch, caches):
         M, dt, f32 = x.shape[0], x.dtype, torch.float32
         proj = self.in_proj(x, GEMM_STORE_F32, out=s.get("proj", f32, M, self.n_proj))
         q = s.get("aq", f32, M, self.col_k)
-        ops.mix_attn_prep(proj, 0, self.col_k, self.col_v, self.bias, self.q_norm_w, self.k_norm_w, self.eps, self.rates, len(self.rate_values),
+        kept = None if self.values == "own" else s.get("v_first", f32, M, self.kv_heads * self.vdim)
+        ops.row_attn_prep(proj, 0, self.col_k, self.col_v, self.bias, self.q_norm_w, self.k_norm_w, self.eps, self.rates, len(self.rate_values),
                           self.mag, self.pairs, self.scale, q, st.keys, st.values, plan["t_row"], plan["t_pos"], self.heads, self.kv_heads,
-                          self.dim, self.vdim)
+                          self.dim, self.vdim, self.temp_coef, self.temp_every, v_first=kept if self.values == "blend" else None,
+                          v_lambda=self.value_mix, v_keep=kept if self.values == "first" else None)
         mix = s.get("mix", dt, M, self.n_mix)
-        ops.mix_attn(q, st.keys, st.values, plan["t_row"], plan["t_pos"], self.talk, self.sink, mix, self.heads, self.kv_heads, self.dim,
-                     self.vdim, window=self.window, cu=plan["cu"], rows=plan["rows"], nb=plan["nb"], max_n=plan["max_n"],
-                     workspace=s.flat("attn_ws", f32) if dt != f32 else None)
+        self.attend(q, st, mix, plan, s.flat("attn_ws", f32) if dt != f32 else None)
         return self.o_proj(mix, GEMM_STORE_F32, out=y_out)
+
+
+class HeadMixAttention(RowNormAttention):
+    """RowNormAttention whose heads' scores are mixed before the softmax: score_h = sum_g talk[h, g] (q_g . k_g * scale); with
+    ``window`` > 0 position i sees j with 0 <= i - j < window."""
+
+    def __init__(self, width: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float, rates: Sequence[float] = (),
+                 mag: float = 1.0, pairs: bool = False, window: int = 0, bias: bool = True, row_norm: bool = True, sink: bool = True):
+        super().__init__(width, heads, kv_heads, dim, vdim, scale, eps, rates, mag, pairs, bias, row_norm, sink)
+        self.window = int(window)
+        self.talk = None                                      # fp32 [heads, heads] on the device
+
+    def workspace_floats(self, rows: int) -> int:
+        return ops.mix_attn_workspace_floats(rows, self.heads, self.vdim)
+
+    def attend(self, q, st: BatchedKVCache, mix, plan: dict, workspace):
+        ops.mix_attn(q, st.keys, st.values, plan["t_row"], plan["t_pos"], self.talk, self.sink, mix, self.heads, self.kv_heads, self.dim,
+                     self.vdim, window=self.window, cu=plan["cu"], rows=plan["rows"], nb=plan["nb"], max_n=plan["max_n"], workspace=workspace)
 
 
 class GatedFF:
@@ -730,12 +766,13 @@ class ActivatedFF:
 
 class RoutedExperts:
     """Mixture of ``experts`` GatedFF experts of which every token uses ``top``; y = sum of the chosen experts' weighted
-    outputs, plus a shared expert (``shared_ff`` > 0) that every token uses.  Two ways to choose (``scoring``):
+    outputs, plus a shared expert (``shared_ff`` > 0) that every token uses.  Ways to choose (``scoring``):
       "softmax"  router logits W_r x + b in fp32, the ``top`` largest chosen, their weights the softmax over the chosen logits;
       "sigmoid"  scores s = sigmoid(W_r x); experts are picked by s + correction (a vector per layer) among the experts of the
                  ``groups[1]`` best of ``groups[0]`` equal groups of neighbouring experts (a group's score: the sum of its two
                  largest picking scores); weights s / sum(chosen s) * ``route_scale``.
-      "scores"   the ``top`` largest s = sigmoid(W_r x) chosen, their weights those scores as they are;
+      "scores"   the ``top`` largest s = sigmoid(W_r x) chosen, their weights those scores as they are or (``renorm``) over their
+                 sum; with ``groups`` only experts of the groups[1] best of groups[0] groups (a group's score: its largest score);
       "softmax_scores"  the same with s = softmax(W_r x) over all experts.
     ``weight_on`` "input": the weight multiplies what the expert reads, y = sum expert_k(w_k x), instead of its output.
     ``limit``: the clamp of experts with the "clamped" unit.
@@ -746,13 +783,13 @@ class RoutedExperts:
 
     def __init__(self, width: int, experts: int, top: int, ff: int, act: str, shared_ff: int = 0, shared_act: Optional[str] = None,
                  router_bias: bool = True, scoring: str = "softmax", groups: Sequence[int] = (1, 1), route_scale: float = 1.0,
-                 shared_gate: bool = False, weight_on: str = "output", limit: float = 0.0):
+                 shared_gate: bool = False, weight_on: str = "output", limit: float = 0.0, renorm: bool = False):
         if scoring not in ("softmax", "sigmoid", "scores", "softmax_scores"):
             raise ValueError(f"unknown expert scoring {scoring!r}")
         if weight_on not in ("output", "input"):
             raise ValueError(f"the routing weight goes on the experts' output or input, not {weight_on!r}")
         self.width, self.experts, self.top, self.ff = width, experts, top, ff
-        self.weight_on, self.limit = weight_on, float(limit)
+        self.weight_on, self.limit, self.renorm = weight_on, float(limit), bool(renorm)
         self.scoring, self.groups, self.route_scale = scoring, (int(groups[0]), int(groups[1])), float(route_scale)
         self.shared_gate = bool(shared_gate and shared_ff)
         self.epilogue = GatedFF.EPILOGUES[act]
@@ -795,7 +832,7 @@ class RoutedExperts:
         seg = s.flat("moe_seg", i32)
         if self.scoring in ("scores", "softmax_scores"):
             ops.moe_route_scores(logits, ids, wts, seg, slot_of, token_of, self.top, experts=self.experts,
-                                 softmax=self.scoring == "softmax_scores")
+                                 softmax=self.scoring == "softmax_scores", groups=self.groups[0], keep=self.groups[1], renorm=self.renorm)
         elif self.scoring == "sigmoid":
             ops.moe_route_sigmoid(logits, self.router_bias, ids, wts, seg, slot_of, token_of, self.top, self.groups[0], self.groups[1],
                                   self.route_scale, experts=self.experts)
@@ -857,8 +894,9 @@ class Sublayer:
 
 
 class LayerRun:
-    """One execution of a layer of the "parallel", the "prenorm" or the "postnorm" chain.  "parallel": x <- x + mixer(n(x)) + mlp(n(x)) with ONE
-    norm n (weight ``norm_w``, fp32, applied as a plain factor).  "prenorm": x <- x + mixer(n(x)), then x <- x + mlp(n2(x)) with a
+    """One execution of a layer of the "parallel", the "prenorm" or the "postnorm" chain.  "parallel": x <- x + m (s1 mixer(n(x)) + s2 mlp(n2(x)))
+    with the norm n (weight ``norm_w``, fp32, applied as a plain factor) and n2 the same norm or (``norm2_w``) one of its own; m is
+    ``SequenceModel.residual_mult``, s1 / s2 the vectors ``scale1`` / ``scale2`` (fp32 on the device; None: ones).  "prenorm": x <- x + mixer(n(x)), then x <- x + mlp(n2(x)) with a
     second norm (``norm2_w``).  ``slot`` is the run's entry in the cache list: a layer that runs several times (a looped span)
     has one run and one state per pass on the same modules.  ``opens``: the run is the first of a pass of the span, which
     begins with x <- W_in [x ; embedding] (``SequenceModel.loop_in``; models without it leave every ``opens`` False).
@@ -872,6 +910,8 @@ class LayerRun:
         self.port2: Optional[StreamPort] = None
         self.norm_w: Optional[torch.Tensor] = None
         self.norm2_w: Optional[torch.Tensor] = None
+        self.scale1: Optional[torch.Tensor] = None
+        self.scale2: Optional[torch.Tensor] = None
         self.avg_w: Optional[torch.Tensor] = None
 
 
@@ -907,7 +947,7 @@ class SequenceModel:
     ``self.final_tanh_norm`` = (alpha, w, b)) and a convolution of ``self.canon_taps`` taps on every sublayer's input;
     "postnorm": ``self.runs`` whose norms stand on the sublayers' outputs, with ``self.embed_norm_w`` (a norm on the embedding) and
     per-run averages over depth as options.
-    ``self.logit_scale`` multiplies the logits."""
+    ``self.logit_scale`` multiplies the logits; ``self.logit_cap`` > 0: logits are cap tanh(logits / cap)."""
 
     block_style = "sandwich"
 
@@ -933,6 +973,10 @@ class SequenceModel:
         self.lm_head: Optional[Linear] = None
         self.eps = 1e-6
         self.logit_scale = 1.0
+        self.logit_cap = 0.0
+        self.residual_mult = 1.0                      # "parallel" chain: multiplies what a run adds to the stream
+        self.overlap_branches = False                 # "parallel" chain: decode steps run a run's two branches side by side
+        self._side: Optional[torch.cuda.Stream] = None
         self.streams, self.canon_taps = 1, 1          # "hyper" chain
         self.embed_norm_w: Optional[torch.Tensor] = None      # "postnorm" chain: norm of the embedding (None: not normed)
         self.depth_average = False                    # "postnorm" chain: the runs have ``avg_w``
@@ -1003,6 +1047,8 @@ class SequenceModel:
                 if r.mlp is not None:
                     r.mlp.reserve(s, dt)
                     s.reserve("y2", torch.float32, W)
+                if self.block_style == "parallel" and r.norm2_w_name is not None:
+                    s.reserve("x2", dt, W)
             if self.loop_in is not None:
                 s.reserve("cat", dt, 2 * W)
             if self.block_style == "hyper":
@@ -1075,35 +1121,59 @@ class SequenceModel:
                 self.residual_tap(sl.layer, sl.kind, h)
 
     def _chain_parallel(self, h, x, y, plan: dict, s: Scratch, cache: List[RowState], M: int):
-        """The runs of a "parallel" model over the residual stream h (fp32): every run reads x = n(h) and adds its branches to h
-        in one pass over the rows, which also prepares what comes next: the next run's normed input, or (before a pass of a
-        looped span) the storage-type copy of h that W_in multiplies beside the embedding."""
+        """The runs of a "parallel" model over the residual stream h (fp32): every run reads x = n(h) (its feed-forward n2(h) where
+        it has a norm of its own) and adds its branches to h in one pass over the rows, which also prepares what comes next: the
+        next run's normed inputs, or (before a pass of a looped span) the storage-type copy of h that W_in multiplies beside the
+        embedding.  With ``overlap_branches`` the two branches of a decode step, which do not depend on each other, are issued to two
+        streams (two chains of a captured graph): both are far too small to fill the GPU."""
         dt, W, eps, runs = self.dtype, self.args.width, self.eps, self.runs
         cat = s.get("cat", dt, M, 2 * W) if self.loop_in is not None else None
+        overlap = self.overlap_branches and plan["max_n"] == 1
+
+        def inputs(r: LayerRun) -> dict:
+            two = dict(w_next2=r.norm2_w, x_out2=s.get("x2", dt, M, W)) if r.norm2_w is not None else {}
+            return dict(w_next=r.norm_w, x_out=x, **two)
 
         def close(i_next: int, y1, y2):
             nxt = runs[i_next] if i_next < len(runs) else None
+            kw = {}
+            if i_next > 0:
+                prev = runs[i_next - 1]
+                kw = dict(y1=y1, y2=y2, c1=self.residual_mult, c2=self.residual_mult, s1=prev.scale1, s2=prev.scale2)
             if nxt is None:
-                if y1 is not None:
-                    ops.residual_add_norm(h, eps, dt, y1=y1, y2=y2)
+                if kw:
+                    ops.residual_add_norm(h, eps, dt, **kw)
             elif nxt.opens:
-                ops.residual_add_norm(h, eps, dt, y1=y1, y2=y2, raw_out=cat[:, :W])
+                ops.residual_add_norm(h, eps, dt, raw_out=cat[:, :W], **kw)
             else:
-                ops.residual_add_norm(h, eps, dt, y1=y1, y2=y2, w_next=nxt.norm_w, x_out=x)
+                ops.residual_add_norm(h, eps, dt, **inputs(nxt), **kw)
             if i_next > 0 and self.residual_tap is not None:
                 self.residual_tap(runs[i_next - 1].layer, "run", h)
             if nxt is not None and nxt.opens:
                 self.loop_in(cat, GEMM_STORE_F32, out=h)
-                ops.residual_add_norm(h, eps, dt, w_next=nxt.norm_w, x_out=x)
+                ops.residual_add_norm(h, eps, dt, **inputs(nxt))
 
         if cat is not None:
             ops.residual_add_norm(h, eps, dt, raw_out=cat[:, W:])           # the embedding, for every pass
         close(0, None, None)
         for i, r in enumerate(runs):
-            r.mixer(x, y, cache[r.slot], plan, s, cache)
-            y2 = None
-            if r.mlp is not None:
-                y2 = r.mlp(x, s.get("y2", torch.float32, M, W), s)
+            if r.mlp is None:
+                r.mixer(x, y, cache[r.slot], plan, s, cache)
+                close(i + 1, y, None)
+                continue
+            x_ff, y2 = s.get("x2", dt, M, W) if r.norm2_w is not None else x, s.get("y2", torch.float32, M, W)
+            if overlap:
+                main = torch.cuda.current_stream(self.device)
+                if self._side is None:
+                    self._side = torch.cuda.Stream(self.device)
+                self._side.wait_stream(main)
+                with torch.cuda.stream(self._side):
+                    r.mlp(x_ff, y2, s)
+                r.mixer(x, y, cache[r.slot], plan, s, cache)
+                main.wait_stream(self._side)
+            else:
+                r.mixer(x, y, cache[r.slot], plan, s, cache)
+                r.mlp(x_ff, y2, s)
             close(i + 1, y, y2)
 
     def _chain_prenorm(self, h, x, y, plan: dict, s: Scratch, cache: List[RowState]):
@@ -1205,7 +1275,10 @@ class SequenceModel:
             ops.tanh_norm(h_rows, *self.final_tanh_norm, xl)
         else:
             ops.norm_add_norm(h_rows, self.eps, self.dtype, w_next=self.final_norm_w, x_out=xl)
-        logits = self.lm_head(xl, GEMM_STORE_F32, out=logits_out)
+        if self.logit_cap:
+            logits = self.lm_head(xl, GEMM_CAP_F32, out=logits_out, act=(self.logit_cap, 0.0))
+        else:
+            logits = self.lm_head(xl, GEMM_STORE_F32, out=logits_out)
         if self.logit_scale != 1.0:
             ops.scale_(logits, self.logit_scale)
         return logits

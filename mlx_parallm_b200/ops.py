@@ -255,7 +255,8 @@ def gemm(x, w, epilogue=_lib.GEMM_STORE, out=None, act=(0.0, 0.0), batch=1, stri
          ldx=None, ldw=None, ldy=None):
     """y = x . w^T with fp32 accumulation (b200p_gemm).  Plain call: x [M, K], w [N, K] of one dtype.  Batched call (one
     weight block per head): pass M, N, K, the row strides and ``strides`` = element strides of x, w, y between products.
-    ``act``: the epilogue's constants (the clamp of GEMM_GLU_CLAMP, the two factors of GEMM_XIELU)."""
+    ``act``: the epilogue's constants (the clamp of GEMM_GLU_CLAMP, the two factors of GEMM_XIELU,
+    the cap of GEMM_CAP_F32)."""
     _dev(x, w, out)
     assert x.dtype == w.dtype and x.stride(-1) == 1 and w.stride(-1) == 1
     if M is None:
@@ -265,10 +266,10 @@ def gemm(x, w, epilogue=_lib.GEMM_STORE, out=None, act=(0.0, 0.0), batch=1, stri
         ldx, ldw = x.stride(0), w.stride(0)
     if out is None:
         n_out = N // 2 if _lib.gemm_is_gated(epilogue) else N
-        out = torch.empty((M, n_out * batch), dtype=torch.float32 if epilogue == _lib.GEMM_STORE_F32 else x.dtype, device=x.device)
+        out = torch.empty((M, n_out * batch), dtype=torch.float32 if _lib.gemm_is_f32(epilogue) else x.dtype, device=x.device)
     if ldy is None:
         ldy = out.stride(0)
-    want = torch.float32 if epilogue == _lib.GEMM_STORE_F32 else x.dtype
+    want = torch.float32 if _lib.gemm_is_f32(epilogue) else x.dtype
     assert out.dtype == want and out.stride(-1) == 1, (out.dtype, want)
     _call(("b200p_gemm", N, K, batch), lambda: lib().b200p_gemm(_p(x), _p(w), _p(out), M, N, K, ldx, ldw, ldy, batch, strides[0], strides[1],
                                                         strides[2], dtype_code(x.dtype), epilogue, float(act[0]), float(act[1]), _stream()))
@@ -371,7 +372,7 @@ def gemm_grouped(x, w, seg, max_rows: int, epilogue=_lib.GEMM_STORE, out=None, a
     groups, N, K = w.shape
     assert x.dtype == w.dtype and x.stride(-1) == 1 and w.is_contiguous() and x.shape[1] == K and seg.dtype == torch.int32
     glu = _lib.gemm_is_gated(epilogue)
-    want = torch.float32 if epilogue == _lib.GEMM_STORE_F32 else x.dtype
+    want = torch.float32 if _lib.gemm_is_f32(epilogue) else x.dtype
     if out is None:
         out = torch.empty((x.shape[0], N // 2 if glu else N), dtype=want, device=x.device)
     assert out.dtype == want and out.stride(-1) == 1
@@ -381,18 +382,21 @@ def gemm_grouped(x, w, seg, max_rows: int, epilogue=_lib.GEMM_STORE, out=None, a
     return out
 
 
-def residual_add_norm(h, eps, dtype, y1=None, c1=1.0, y2=None, c2=1.0, w_next=None, x_out=None, raw_out=None):
-    """h += c1 y1 + c2 y2; raw_out = h (may be a column slice); x_out = rms_norm(h) * w_next (b200p_residual_add_norm)."""
-    _dev(h, y1, y2, w_next, x_out, raw_out)
+def residual_add_norm(h, eps, dtype, y1=None, c1=1.0, y2=None, c2=1.0, w_next=None, x_out=None, raw_out=None, s1=None, s2=None,
+                      w_next2=None, x_out2=None):
+    """h += c1 s1 y1 + c2 s2 y2 (s1, s2: fp32 [W], None: ones); raw_out = h (may be a column slice); x_out = rms_norm(h) * w_next,
+    x_out2 = rms_norm(h) * w_next2 (b200p_residual_add_norm)."""
+    _dev(h, y1, y2, w_next, x_out, raw_out, s1, s2, w_next2, x_out2)
     M, W = h.shape
     assert h.dtype == torch.float32 and h.is_contiguous()
-    for t in (y1, y2, w_next):
+    for t in (y1, y2, w_next, s1, s2, w_next2):
         assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
-    assert x_out is None or (x_out.dtype == dtype and x_out.is_contiguous())
+    for t in (x_out, x_out2):
+        assert t is None or (t.dtype == dtype and t.is_contiguous())
     assert raw_out is None or (raw_out.dtype == dtype and raw_out.stride(1) == 1)
     _call("b200p_residual_add_norm", lambda: lib().b200p_residual_add_norm(
-        _p(h), _p(y1), float(c1), _p(y2), float(c2), _p(w_next), _p(x_out), _p(raw_out), 0 if raw_out is None else raw_out.stride(0), M, W,
-        float(eps), dtype_code(dtype), _stream()))
+        _p(h), _p(y1), float(c1), _p(s1), _p(y2), float(c2), _p(s2), _p(w_next), _p(x_out), _p(w_next2), _p(x_out2), _p(raw_out),
+        0 if raw_out is None else raw_out.stride(0), M, W, float(eps), dtype_code(dtype), _stream()))
 
 
 def cast_columns(src, dst):
@@ -617,14 +621,17 @@ def window_attn(q, kcache, vcache, t_row, t_pos, out, H, G, dk, dv, softcap=0.0,
     return out
 
 
-def moe_route_scores(logits, ids, wts, seg, slot_of, token_of, top: int, experts: Optional[int] = None, softmax: bool = False):
-    """Routing by the largest sigmoid scores, or the largest of a softmax over all experts; the weights are the scores themselves."""
+def moe_route_scores(logits, ids, wts, seg, slot_of, token_of, top: int, experts: Optional[int] = None, softmax: bool = False,
+                     groups: int = 1, keep: int = 1, renorm: bool = False):
+    """Routing by the largest sigmoid scores, or the largest of a softmax over all experts, inside the ``keep`` best of ``groups``
+    expert groups (a group counts as its best expert); the weights are the scores themselves, or (``renorm``) their shares."""
     _dev(logits, ids, wts, seg, slot_of, token_of)
     M = logits.shape[0]
     E = logits.shape[1] if experts is None else int(experts)
     assert logits.dtype == torch.float32 and logits.stride(1) == 1
     _call("b200p_moe_route_scores", lambda: lib().b200p_moe_route_scores(_p(logits), logits.stride(0), _p(ids), _p(wts), _p(seg), _p(slot_of),
-                                                                        _p(token_of), M, E, int(top), int(softmax), _stream()))
+                                                                        _p(token_of), M, E, int(top), int(softmax), int(groups), int(keep),
+                                                                        int(renorm), _stream()))
 
 
 def moe_scatter_scaled(x, slot_of, wts, xs, top: int):
@@ -690,19 +697,22 @@ def post_norm_step(h, w, eps, dtype, y=None, stack=None, slot=-1, avg=None, raw_
         _p(raw_out), M, W, float(eps), dtype_code(dtype), _stream()))
 
 
-def mix_attn_prep(proj, col_q, col_k, col_v, bias, wq, wk, eps, rates, n_rot, mag, pairs, scale, q_out, kcache, vcache, t_row, t_pos, H, G,
-                  dk, dv):
-    """Biased, normed (whole rows), rotated, scaled queries to ``q_out`` fp32 [M, H dk]; keys and values into the caches
-    [rows, G, Tcap, dk] / [rows, G, Tcap, dv] at every token's (row, position)."""
-    _dev(proj, bias, wq, wk, rates, q_out, kcache, vcache, t_row, t_pos)
+def row_attn_prep(proj, col_q, col_k, col_v, bias, wq, wk, eps, rates, n_rot, mag, pairs, scale, q_out, kcache, vcache, t_row, t_pos, H, G,
+                  dk, dv, temp_coef=0.0, temp_every=1.0, v_first=None, v_lambda=0.0, v_keep=None):
+    """Biased, normed (whole rows), rotated, tempered, scaled queries to ``q_out`` fp32 [M, H dk]; keys and values into the caches
+    [rows, G, Tcap, dk] / [rows, G, Tcap, dv] at every token's (row, position).  ``v_first`` fp32 [M, G dv]: values are
+    (1 - v_lambda) v + v_lambda v_first; ``v_keep`` fp32 [M, G dv] receives them."""
+    _dev(proj, bias, wq, wk, rates, q_out, kcache, vcache, t_row, t_pos, v_first, v_keep)
     M = proj.shape[0]
     assert proj.dtype == torch.float32 and proj.stride(1) == 1 and kcache.is_contiguous() and vcache.is_contiguous() and q_out.is_contiguous()
     assert kcache.dtype == vcache.dtype and kcache.shape[1:] == (G, kcache.shape[2], dk) and vcache.shape[1:] == (G, kcache.shape[2], dv)
     assert (wq is None or wq.numel() == H * dk) and (wk is None or wk.numel() == G * dk) and (n_rot == 0 or rates.numel() == n_rot)
-    _call("b200p_mix_attn_prep", lambda: lib().b200p_mix_attn_prep(
+    for t in (v_first, v_keep):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.shape == (M, G * dv))
+    _call("b200p_row_attn_prep", lambda: lib().b200p_row_attn_prep(
         _p(proj), proj.stride(0), int(col_q), int(col_k), int(col_v), _p(bias), _p(wq), _p(wk), float(eps), _p(rates), int(n_rot), float(mag),
-        int(pairs), float(scale), _p(q_out), _p(kcache), _p(vcache), kcache.shape[2], _p(t_row), _p(t_pos), M, H, G, dk, dv,
-        dtype_code(kcache.dtype), _stream()))
+        int(pairs), float(scale), float(temp_coef), float(temp_every), _p(v_first), float(v_lambda), _p(v_keep), _p(q_out), _p(kcache),
+        _p(vcache), kcache.shape[2], _p(t_row), _p(t_pos), M, H, G, dk, dv, dtype_code(kcache.dtype), _stream()))
 
 
 def mix_attn_workspace_floats(nb: int, H: int, dv: int) -> int:

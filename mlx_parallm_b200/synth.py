@@ -709,3 +709,70 @@ def seradra_random_weights(cfg: dict, seed: int = 1234, device="cpu") -> Dict[st
             t = 1.0 + r * 0.02
         out[name] = t.to(torch.bfloat16)
     return out
+
+
+# ---- Negosun ----------------------------------------------------------------------------------------------------------------
+def negosun_config(width: int, ff: int, n_layers: int, heads: int, head_dim: int, kv_heads: Optional[int] = None, experts: int = 16,
+                   top: int = 2, expert_groups: int = 4, keep_groups: int = 2, vocab: int = 32000, **unused) -> dict:
+    """A config of the design at the sizes of a real model: every layer attention beside routed experts; the experts a token uses
+    and the shared expert together have the hidden size ``ff``."""
+    mixer = {"heads": heads, "kv_heads": kv_heads or max(1, heads // 4), "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+             "q_temp": {"coef": 0.1, "every": 512}, "v_mix": True}
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": expert_groups, "keep": keep_groups}},
+           "expert": {"ff": ff // (2 * top)}, "shared": {"ff": ff // 2}}
+    return {"architecture": "Negosun", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_softcap": 30.0,
+            "layers": [{"type": "attention", "mixer": dict(mixer), "mlp": mlp} for _ in range(n_layers)]}
+
+
+def negosun_shapes(cfg: dict) -> Dict[str, tuple]:
+    """Shape of every tensor of a Negosun checkpoint (matrices [out, in])."""
+    W, V = cfg["width"], cfg["vocab"]
+    out = {"embed": (V, W), "final.norm": (W,)}
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.mix.", L["mixer"]
+        H = m["heads"]
+        G = m.get("kv_heads", H)
+        out[f"l{i}.norm1"] = out[f"l{i}.ls1"] = (W,)
+        for n, rows in (("q", H * m["dim"]), ("k", G * m["dim"]), ("v", G * m["vdim"])):
+            out[p + n], out[f"{p}{n}.b"] = (rows, W), (rows,)
+            if n != "v":
+                out[f"{p}{n}.norm"] = (rows,)
+        out[p + "o"] = (W, H * m["vdim"])
+        if m.get("v_mix"):
+            out[p + "vmix"] = ()
+        mlp = L.get("mlp")
+        if mlp is None:
+            continue
+        q = f"l{i}.mlp."
+        out[f"l{i}.norm2"] = out[f"l{i}.ls2"] = (W,)
+        parts = {f"{q}e{e}.": mlp["expert"]["ff"] for e in range(mlp["router"]["experts"])}
+        if mlp.get("shared"):
+            parts[q + "shared."] = mlp["shared"]["ff"]
+        for pre, n in parts.items():
+            out[pre + "gate"] = out[pre + "up"] = (n, W)
+            out[pre + "down"] = (W, n)
+        out[q + "router"] = (mlp["router"]["experts"], W)
+    return out
+
+
+def negosun_random_weights(cfg: dict, seed: int = 1234, device="cpu") -> Dict[str, torch.Tensor]:
+    """bfloat16 tensors: matrices N(0, 1/in), norm weights and channel scales near one, biases small, value mixing near a half."""
+    dev = torch.device(device)
+    out: Dict[str, torch.Tensor] = {}
+    for name, shape in negosun_shapes(cfg).items():
+        g = torch.Generator(device=dev)
+        g.manual_seed(_stable_seed(seed, name))
+        r = torch.randn(shape, generator=g, device=dev)
+        leaf = name.split(".")[-1]
+        if name == "embed":
+            t = r
+        elif len(shape) == 2:
+            t = r / math.sqrt(shape[1])
+        elif leaf == "b":
+            t = r * 0.1
+        elif leaf == "vmix":
+            t = 0.5 + r * 0.1
+        else:
+            t = 1.0 + r * 0.02
+        out[name] = t.to(torch.bfloat16)
+    return out

@@ -213,7 +213,7 @@ def test_attention_preparation(H, G, d, dv, n_rot, pairs, bias, normed):
     rates, mag = O.rates_of({"dims": 2 * n_rot, "base": 300.0, "scaling": {"factor": 6.0, "original": 40, "fast": 8.0, "slow": 0.5}})
     q = torch.zeros(M, H * d, device="cuda")
     kc, vc = torch.full((2, G, 5001, d), 5.0, device="cuda"), torch.full((2, G, 5001, dv), 5.0, device="cuda")
-    ops.mix_attn_prep(proj.cuda(), 0, H * d, (H + G) * d, bv.cuda() if bias else None, wq.cuda() if normed else None,
+    ops.row_attn_prep(proj.cuda(), 0, H * d, (H + G) * d, bv.cuda() if bias else None, wq.cuda() if normed else None,
                       wk.cuda() if normed else None, 1e-3, torch.tensor(rates, dtype=torch.float32, device="cuda") if rates else None, n_rot,
                       mag, pairs, 0.3, q, kc, vc, torch.ones(M, **I32), torch.tensor(pos, **I32), H, G, d, dv)
     p = proj[:, :n].double() + (bv.double() if bias else 0.0)
