@@ -396,13 +396,20 @@ static int gemm_dispatch(const void* x, const void* w, void* y, int64_t M, int64
   return B200P_OK;
 }
 
-// groups of at most max_rows rows each: the row-streaming kernel while a group fits its 64 rows, 64 x 64 tiles beyond
+// groups of at most max_rows rows each: tcgen05 where it takes the shape, else the row-streaming kernel while a group fits its 64 rows
+// and 64 x 64 tiles beyond
 template <typename T>
 static int gemm_grouped_dispatch(const void* x, const void* w, void* y, const int32_t* seg, int64_t total_rows, int64_t max_rows, int64_t N, int64_t K,
                                  int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t sw, int epi, float2 act, bool fast_ok,
                                  cudaStream_t st) {
   const T* xp = (const T*)x;
   const T* wp = (const T*)w;
+  if constexpr (!std::is_same<T, float>::value) {
+    if (fast_ok && g_gemm_path != 1) {
+      const int rc = gemm_tc_launch_grouped<T>(xp, wp, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, sw, epi, act, st);
+      if (rc != 1) return rc;
+    }
+  }
   if (fast_ok && max_rows <= 64) {
     dim3 grid((unsigned)((N + 15) / 16), 1, (unsigned)groups);
     if (max_rows <= 16) gemm_stream_kernel<T, 1><<<grid, GK_THREADS, 0, st>>>(xp, wp, y, 0, N, K, ldx, ldw, ldy, 0, sw, 0, epi, act, seg);
@@ -412,12 +419,6 @@ static int gemm_grouped_dispatch(const void* x, const void* w, void* y, const in
     return B200P_OK;
   }
   if (fast_ok) {
-    if constexpr (!std::is_same<T, float>::value) {
-      if (g_gemm_path != 1) {
-        const int rc = gemm_tc_launch_grouped<T>(xp, wp, y, seg, total_rows, max_rows, N, K, ldx, ldw, ldy, groups, sw, epi, act, st);
-        if (rc != 1) return rc;
-      }
-    }
     return gemm_mma_launch<T, 2, 2, 32, 32, 32, 3>(xp, wp, y, max_rows, N, K, ldx, ldw, ldy, groups, 0, sw, 0, epi, act, st, seg);
   }
   dim3 grid((unsigned)((N + GS_BN - 1) / GS_BN), (unsigned)((max_rows + GS_BM - 1) / GS_BM), (unsigned)groups);

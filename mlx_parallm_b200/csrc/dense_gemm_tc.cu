@@ -47,8 +47,8 @@ struct GemmTcParams {
   int trans;                     // operands swapped: accumulator row = output column, accumulator column = token
   int epi, vec_ok;
   float2 act;
-  // grouped products (not with trans): batch index z owns the rows [seg[z], seg[z+1]) of x and y; tiles past a group's rows are
-  // skipped by every role alike; seg (device, groups + 1 offsets) is copied to shared memory first
+  // grouped products: batch index z owns the rows [seg[z], seg[z+1]) of x and y; tiles past a group's rows (with trans: tiles of a
+  // group without rows) are skipped by every role alike; seg (device, groups + 1 offsets) is copied to shared memory first
   const int32_t* seg;
   int groups;
 };
@@ -152,14 +152,15 @@ __device__ __forceinline__ void gemm_tc_store32(const GemmTcParams& p, int64_t r
 }
 
 // Swapped operands: this thread owns output column `n` (a weight row) and holds it for 32 consecutive tokens from `tok0`.
-// p.M counts output columns and p.N tokens here.  Gate / up pairs sit in neighbouring lanes.
+// p.M counts output columns here; `tokens` of this batch index (group) exist.  Gate / up pairs sit in neighbouring lanes.
 template <typename T>
-__device__ __forceinline__ void gemm_tc_store32_trans(const GemmTcParams& p, int64_t z_off, int64_t n, int64_t tok0, const float (&v)[32]) {
+__device__ __forceinline__ void gemm_tc_store32_trans(const GemmTcParams& p, int64_t z_off, int64_t n, int64_t tok0, int64_t tokens,
+                                                      const float (&v)[32]) {
   if (gemm_epi_is_glu(p.epi)) {
 #pragma unroll
     for (int i = 0; i < 32; ++i) {
       const float other = __shfl_xor_sync(0xffffffffu, v[i], 1);
-      if (!(threadIdx.x & 1) && n + 1 < p.M && tok0 + i < p.N)
+      if (!(threadIdx.x & 1) && n + 1 < p.M && tok0 + i < tokens)
         reinterpret_cast<T*>(p.y)[z_off + (tok0 + i) * p.ldy + (n >> 1)] = Tr<T>::from_f(glu_unit(v[i], other, p.epi, p.act));
     }
     return;
@@ -170,22 +171,22 @@ __device__ __forceinline__ void gemm_tc_store32_trans(const GemmTcParams& p, int
     if (p.splits > 1) {
 #pragma unroll
       for (int i = 0; i < 32; ++i)
-        if (tok0 + i < p.N) atomicAdd(dst + (tok0 + i) * p.ldy, v[i]);
+        if (tok0 + i < tokens) atomicAdd(dst + (tok0 + i) * p.ldy, v[i]);
     } else {
 #pragma unroll
       for (int i = 0; i < 32; ++i)
-        if (tok0 + i < p.N) dst[(tok0 + i) * p.ldy] = v[i];
+        if (tok0 + i < tokens) dst[(tok0 + i) * p.ldy] = v[i];
     }
   } else if (p.epi == B200P_GEMM_CAP_F32) {
     float* dst = reinterpret_cast<float*>(p.y) + z_off + n;
 #pragma unroll
     for (int i = 0; i < 32; ++i)
-      if (tok0 + i < p.N) dst[(tok0 + i) * p.ldy] = gemm_f32_act(v[i], p.epi, p.act);
+      if (tok0 + i < tokens) dst[(tok0 + i) * p.ldy] = gemm_f32_act(v[i], p.epi, p.act);
   } else {
     T* dst = reinterpret_cast<T*>(p.y) + z_off + n;
 #pragma unroll
     for (int i = 0; i < 32; ++i)
-      if (tok0 + i < p.N) dst[(tok0 + i) * p.ldy] = Tr<T>::from_f(gemm_store_act(v[i], p.epi, p.act));
+      if (tok0 + i < tokens) dst[(tok0 + i) * p.ldy] = Tr<T>::from_f(gemm_store_act(v[i], p.epi, p.act));
   }
 }
 
@@ -196,14 +197,15 @@ struct GemmTcShared {            // lives behind the ring stages (8-byte aligned
   int seg[GT_MAX_GROUPS + 1];
 };
 
-// rows of group z that tile mt covers: first row in x / y and how many rows the group has; false when the tile is past them
+// rows of group z that tile mt covers: first row in x / y and how many rows the group has; false when the tile is past them (with
+// swapped operands tiles run over the weights, and only a group without rows has none)
 __device__ __forceinline__ bool gemm_tc_group_tile(const GemmTcParams& p, const GemmTcShared* sh, int z, int mt, int& first, int& len) {
   first = 0;
-  len = (int)p.M;
+  len = p.trans ? (int)p.N : (int)p.M;
   if (!p.seg) return true;
   first = sh->seg[z];
   len = sh->seg[z + 1] - first;
-  return mt * GT_BM < len;
+  return p.trans ? len > 0 : mt * GT_BM < len;
 }
 
 // bounded wait: gives up after about a second, or as soon as another role of the CTA has given up
@@ -284,8 +286,13 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmx, const __grid_constant__ 
           const uint32_t bar = smem_u32(&sh->full[stage]);
           const uint32_t dst = base + stage * STAGE_BYTES;
           mbar_arrive_expect_tx(bar, STAGE_BYTES);
-          tma_load_3d(dst, &tmx, kb * GT_BK, first + mt * GT_BM, p.seg ? 0 : z, bar);
-          tma_load_3d(dst + GT_A_BYTES, &tmw, kb * GT_BK, nt * BN, z, bar);
+          if (p.trans) {                            // A = weights, B = tokens
+            tma_load_3d(dst, &tmx, kb * GT_BK, mt * GT_BM, z, bar);
+            tma_load_3d(dst + GT_A_BYTES, &tmw, kb * GT_BK, first + nt * BN, p.seg ? 0 : z, bar);
+          } else {
+            tma_load_3d(dst, &tmx, kb * GT_BK, first + mt * GT_BM, p.seg ? 0 : z, bar);
+            tma_load_3d(dst + GT_A_BYTES, &tmw, kb * GT_BK, nt * BN, z, bar);
+          }
           if (++stage == STAGES) { stage = 0; phase ^= 1u; }
         }
       }
@@ -346,7 +353,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmx, const __grid_constant__ 
         tmem_ld16(tsrc + c, *reinterpret_cast<float(*)[16]>(&v[0]));
         tmem_ld16(tsrc + c + 16, *reinterpret_cast<float(*)[16]>(&v[16]));
         tmem_ld_wait();
-        if (p.trans) gemm_tc_store32_trans<T>(p, (int64_t)z * p.sy, row, n0, v);
+        if (p.trans) gemm_tc_store32_trans<T>(p, p.seg ? first * p.ldy : (int64_t)z * p.sy, row, n0, len, v);
         else if (row < len) gemm_tc_store32<T>(p, row_off, n0, v);
       }
       tc_fence_before();
@@ -486,7 +493,8 @@ int gemm_tc_launch(const T* x, const T* w, void* y, int64_t M, int64_t N, int64_
 // Grouped product: x [total_rows, K] holds the groups' rows back to back (group z: rows [seg[z], seg[z+1]), at most max_rows of
 // them), w [groups][N][K].  The tile list covers max_rows rows for every group; tiles past a group's rows cost a shared-memory
 // read.  A tile's 128-row box may reach into the next group's rows (or past the tensor, which reads zeros): those accumulator
-// rows are not stored.
+// rows are not stored.  Groups of at most 64 rows (decode steps) swap the operands: tiles of 128 weight rows against a group's tokens;
+// declined when the groups that can have rows are too few to occupy the SMs.
 template <typename T>
 int gemm_tc_launch_grouped(const T* x, const T* w, void* y, const int32_t* seg, int64_t total_rows, int64_t max_rows, int64_t N,
                            int64_t K, int64_t ldx, int64_t ldw, int64_t ldy, int64_t groups, int64_t sw, int epi, float2 act,
@@ -494,29 +502,32 @@ int gemm_tc_launch_grouped(const T* x, const T* w, void* y, const int32_t* seg, 
   if (K < GT_BK || total_rows >= (1ll << 31) || N >= (1ll << 31) || K >= (1ll << 31) || groups > GT_MAX_GROUPS) return 1;
   TcEncodeFn enc = gemm_tc_encode_fn();
   if (!enc) return 1;
-  const int bn = N <= 64 ? 64 : N <= 128 ? 128 : 256;
+  const bool trans = max_rows <= 64;
+  if (trans && min(groups, total_rows) * ((N + GT_BM - 1) / GT_BM) < sm_count()) return 1;
+  const int bn = trans ? (max_rows <= 32 ? 32 : 64) : N <= 64 ? 64 : N <= 128 ? 128 : 256;
   const CUtensorMapDataType dt = std::is_same<T, __nv_bfloat16>::value ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16;
   CUtensorMap tmx, tmw;
-  if (!gemm_tc_map(enc, &tmx, dt, x, K, total_rows, 1, ldx, 0, GT_BM)) return 1;
-  if (!gemm_tc_map(enc, &tmw, dt, w, K, N, groups, ldw, sw, bn)) return 1;
+  if (!gemm_tc_map(enc, &tmx, dt, x, K, total_rows, 1, ldx, 0, trans ? bn : GT_BM)) return 1;
+  if (!gemm_tc_map(enc, &tmw, dt, w, K, N, groups, ldw, sw, trans ? GT_BM : bn)) return 1;
   GemmTcParams p;
   p.y = y;
-  p.M = max_rows; p.N = N; p.K = K; p.ldy = ldy; p.sy = 0;
-  p.tiles_m = (int)((max_rows + GT_BM - 1) / GT_BM);
-  p.tiles_n = (int)((N + bn - 1) / bn);
+  p.M = trans ? N : max_rows; p.N = trans ? max_rows : N; p.K = K; p.ldy = ldy; p.sy = 0;
+  p.tiles_m = (int)((p.M + GT_BM - 1) / GT_BM);
+  p.tiles_n = (int)((p.N + bn - 1) / bn);
   const int64_t nt = (int64_t)p.tiles_m * p.tiles_n * groups;
   if (nt >= (1ll << 31)) return 1;
   p.num_tiles = (int)nt;
   p.num_kb = (int)((K + GT_BK - 1) / GT_BK);
   p.splits = 1;
   p.kb_per_split = p.num_kb;
-  p.trans = 0;
+  p.trans = trans;
   p.seg = seg;
   p.groups = (int)groups;
   p.epi = epi;
   p.act = act;
   const int64_t eb = (epi == B200P_GEMM_STORE_F32 || epi == B200P_GEMM_CAP_F32) ? 4 : 2;
   p.vec_ok = aligned(y, 16) && (ldy * eb) % 16 == 0;
+  if (trans) return bn == 32 ? gemm_tc_run<T, 32, 10>(tmw, tmx, p, st) : gemm_tc_run<T, 64, 8>(tmw, tmx, p, st);
   if (bn == 256) return gemm_tc_run<T, 256, 4>(tmx, tmw, p, st);
   if (bn == 128) return gemm_tc_run<T, 128, 6>(tmx, tmw, p, st);
   return gemm_tc_run<T, 64, 8>(tmx, tmw, p, st);

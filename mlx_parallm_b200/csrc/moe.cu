@@ -209,6 +209,8 @@ __global__ void moe_scatter_scaled_kernel(const T* __restrict__ x, const int32_t
   for (int64_t c = threadIdx.x; c < W; c += blockDim.x) dst[c] = Tr<T>::from_f(w * Tr<T>::to_f(src[c]));
 }
 
+// V neighbouring channels per access (4: rows of whole 16-byte pieces)
+template <int V>
 __global__ void moe_combine_kernel(const float* __restrict__ ye, const int32_t* __restrict__ slot_of, const float* __restrict__ wts,
                                    const float* __restrict__ shared_y, const float* __restrict__ shared_gate, int64_t ldg,
                                    float* __restrict__ y, int64_t W, int top) {
@@ -221,11 +223,23 @@ __global__ void moe_combine_kernel(const float* __restrict__ ye, const int32_t* 
     wt[threadIdx.x] = wts ? wts[t * top + threadIdx.x] : 1.f;
   }
   __syncthreads();
-  for (int64_t c = threadIdx.x; c < W; c += blockDim.x) {
-    float a = 0.f;
-    for (int k = 0; k < top; ++k) a = fmaf(wt[k], ye[(int64_t)sl[k] * W + c], a);
-    if (shared_y) a = fmaf(sg, shared_y[t * W + c], a);
-    y[t * W + c] = a;
+  for (int64_t c = (int64_t)threadIdx.x * V; c < W; c += (int64_t)blockDim.x * V) {
+    float a[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) a[i] = 0.f;
+    auto add = [&](float w, const float* p) {
+      if constexpr (V == 4) {
+        const float4 q = *reinterpret_cast<const float4*>(p);
+        a[0] = fmaf(w, q.x, a[0]); a[1] = fmaf(w, q.y, a[1]); a[2] = fmaf(w, q.z, a[2]); a[3] = fmaf(w, q.w, a[3]);
+      } else {
+        a[0] = fmaf(w, p[0], a[0]);
+      }
+    };
+#pragma unroll 4
+    for (int k = 0; k < top; ++k) add(wt[k], ye + (int64_t)sl[k] * W + c);
+    if (shared_y) add(sg, shared_y + t * W + c);
+    if constexpr (V == 4) *reinterpret_cast<float4*>(y + t * W + c) = make_float4(a[0], a[1], a[2], a[3]);
+    else y[t * W + c] = a[0];
   }
 }
 
@@ -319,7 +333,11 @@ extern "C" int b200p_moe_combine(const float* ye, const int32_t* slot_of, const 
                                  const float* shared_gate, int64_t ldg, float* y, int64_t M, int64_t W, int top, void* stream) {
   B200P_REQUIRE(ye && slot_of && y && W > 0 && top > 0 && top <= MOE_MAX_TOP, B200P_ERR_ARG, "null pointer or bad top");
   if (M == 0) return B200P_OK;
-  moe_combine_kernel<<<(unsigned)M, W >= 1024 ? 256 : 128, 0, (cudaStream_t)stream>>>(ye, slot_of, wts, shared_y, shared_gate, ldg, y, W, top);
+  const unsigned threads = W >= 1024 ? 256 : 128;
+  if (W % 4 == 0 && aligned(ye, 16) && aligned(shared_y, 16) && aligned(y, 16))
+    moe_combine_kernel<4><<<(unsigned)M, threads, 0, (cudaStream_t)stream>>>(ye, slot_of, wts, shared_y, shared_gate, ldg, y, W, top);
+  else
+    moe_combine_kernel<1><<<(unsigned)M, threads, 0, (cudaStream_t)stream>>>(ye, slot_of, wts, shared_y, shared_gate, ldg, y, W, top);
   B200P_LAUNCH_CHECK("moe_combine_kernel");
   return B200P_OK;
 }

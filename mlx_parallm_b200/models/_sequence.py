@@ -1128,7 +1128,7 @@ class SequenceModel:
         streams (two chains of a captured graph): both are far too small to fill the GPU."""
         dt, W, eps, runs = self.dtype, self.args.width, self.eps, self.runs
         cat = s.get("cat", dt, M, 2 * W) if self.loop_in is not None else None
-        overlap = self.overlap_branches and plan["max_n"] == 1
+        overlap = self.overlap_branches and plan["max_n"] == 1 and ops.PROFILER is None      # events around calls time one call each
 
         def inputs(r: LayerRun) -> dict:
             two = dict(w_next2=r.norm2_w, x_out2=s.get("x2", dt, M, W)) if r.norm2_w is not None else {}
