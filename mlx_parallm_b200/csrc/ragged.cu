@@ -148,9 +148,9 @@ __device__ __forceinline__ void load_row(const float* p, float (&v)[V]) {
 // V neighbouring channels per access; the first R pieces of a thread's row stay in registers between the sum of squares and the
 // normed stores, longer rows are read again (by the thread that wrote them).
 template <typename T, int V, int R>
-__global__ void residual_add_norm_kernel(float* __restrict__ h, const float* __restrict__ y1, float c1, const float* __restrict__ s1,
-                                         const float* __restrict__ y2, float c2, const float* __restrict__ s2, ResidualOut out, int64_t W,
-                                         float eps) {
+__global__ void __launch_bounds__(512, 3)            // three rows in flight per SM: one CTA's reduction hides behind the others' loads
+residual_add_norm_kernel(float* __restrict__ h, const float* __restrict__ y1, float c1, const float* __restrict__ s1,
+                         const float* __restrict__ y2, float c2, const float* __restrict__ s2, ResidualOut out, int64_t W, float eps) {
   __shared__ float red[32];
   const int64_t row = blockIdx.x, step = (int64_t)blockDim.x * V;
   float* hr = h + row * W;

@@ -975,7 +975,7 @@ class SequenceModel:
         self.logit_scale = 1.0
         self.logit_cap = 0.0
         self.residual_mult = 1.0                      # "parallel" chain: multiplies what a run adds to the stream
-        self.overlap_branches = False                 # "parallel" chain: decode steps run a run's two branches side by side
+        self.overlap_branches = True                  # "parallel" chain: decode steps run a run's two branches side by side
         self._side: Optional[torch.cuda.Stream] = None
         self.streams, self.canon_taps = 1, 1          # "hyper" chain
         self.embed_norm_w: Optional[torch.Tensor] = None      # "postnorm" chain: norm of the embedding (None: not normed)

@@ -87,7 +87,6 @@ class Model(SequenceModel):
         self.eps = float(args.norm.get("eps", 1e-6))
         self.residual_mult = float(args.residual_mult)
         self.logit_cap = float(args.logit_softcap or 0.0)
-        self.overlap_branches = True
         self.embed = HashedBigramEmbedding(args.vocab, W, 1.0)
         first_mixed = next((i for i, L in enumerate(args.layers) if L["mixer"].get("v_mix")), None)
         for i, L in enumerate(args.layers):
